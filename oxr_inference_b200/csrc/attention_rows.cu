@@ -163,14 +163,16 @@ OXR_API int oxr_scatter_rows(void* pool, long long slot_stride, long long pool_s
 // One block per token. down[t] = [rank compressed | rot shared key part]:
 //   pool[slot] = [ rmsnorm(compressed) * weight | rotate(key part) ]        (skipped for slot -1)
 //   q_out[t, h, qo_rot0 : qo_rot0 + rot] = rotate(q[t, h, q_rot0 : q_rot0 + rot])  for every head (q_out may be q)
-// rotate: entries 2i and 2i+1 of the first 2 * half entries turn by the token's angle i; the rest pass unchanged.
+// rotate: the first 2 * half entries turn by the token's angles, angle i turning entries 2i and 2i+1 or, with `halves`, entries i and i + half;
+// the rest pass unchanged. `down` rows are down_stride apart (columns of a wider product).
 template <typename T>
-__global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, long long pool_slots, const T* __restrict__ down, int rank, int rot,
+__global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, long long pool_slots, const T* __restrict__ down, int down_stride, int rank, int rot,
                                    const float* __restrict__ weight, float eps, const T* q, int heads, int q_head_dim, int q_rot0, T* q_out,
-                                   int qo_head_dim, int qo_rot0, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int half, const int* __restrict__ slots, int* status) {
+                                   int qo_head_dim, int qo_rot0, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int half, int halves, const int* __restrict__ slots, int* status) {
     __shared__ float red[32];
     const int t = blockIdx.x;
-    const T* row = down + (size_t)t * (rank + rot);
+    const int step = halves ? 1 : 2, gap = halves ? half : 1;     // pair i: entries step * i and step * i + gap
+    const T* row = down + (size_t)t * down_stride;
     float ss = 0.f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) {
         const float v = Num<T>::to_f32(row[i]);
@@ -187,9 +189,9 @@ __global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, 
         T* dst = pool + (long long)slot * slot_stride;
         for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = Num<T>::from_f32(Num<T>::to_f32(row[i]) * inv * weight[i]);
         for (int i = threadIdx.x; i < half; i += blockDim.x) {
-            const float u = Num<T>::to_f32(row[rank + 2 * i]), v = Num<T>::to_f32(row[rank + 2 * i + 1]);
-            dst[rank + 2 * i] = Num<T>::from_f32(u * c[i] - v * s[i]);
-            dst[rank + 2 * i + 1] = Num<T>::from_f32(v * c[i] + u * s[i]);
+            const float u = Num<T>::to_f32(row[rank + step * i]), v = Num<T>::to_f32(row[rank + step * i + gap]);
+            dst[rank + step * i] = Num<T>::from_f32(u * c[i] - v * s[i]);
+            dst[rank + step * i + gap] = Num<T>::from_f32(v * c[i] + u * s[i]);
         }
         for (int i = 2 * half + threadIdx.x; i < rot; i += blockDim.x) dst[rank + i] = row[rank + i];
     }
@@ -197,9 +199,9 @@ __global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, 
         const int h = i / half, k = i % half;
         const T* qr = q + ((size_t)t * heads + h) * q_head_dim + q_rot0;
         T* qo = q_out + ((size_t)t * heads + h) * qo_head_dim + qo_rot0;
-        const float u = Num<T>::to_f32(qr[2 * k]), v = Num<T>::to_f32(qr[2 * k + 1]);
-        qo[2 * k] = Num<T>::from_f32(u * c[k] - v * s[k]);
-        qo[2 * k + 1] = Num<T>::from_f32(v * c[k] + u * s[k]);
+        const float u = Num<T>::to_f32(qr[step * k]), v = Num<T>::to_f32(qr[step * k + gap]);
+        qo[step * k] = Num<T>::from_f32(u * c[k] - v * s[k]);
+        qo[step * k + gap] = Num<T>::from_f32(v * c[k] + u * s[k]);
     }
     const int rest = rot - 2 * half;
     if (rest > 0 && q_out != q)
@@ -209,18 +211,41 @@ __global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, 
         }
 }
 
-OXR_API int oxr_latent_prep(void* pool, long long slot_stride, long long pool_slots, const void* down, int rank, int rot, const float* weight, float eps,
+OXR_API int oxr_latent_prep(void* pool, long long slot_stride, long long pool_slots, const void* down, int down_stride, int rank, int rot, const float* weight, float eps,
                             const void* q, int heads, int q_head_dim, int q_rot0, void* q_out, int qo_head_dim, int qo_rot0, const float* cos_t,
-                            const float* sin_t, int half, const int* slots, int n_tokens, int dtype, int* status, cudaStream_t stream) {
+                            const float* sin_t, int half, int halves, const int* slots, int n_tokens, int dtype, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (rank <= 0 || rot < 0 || 2 * half > rot || q_rot0 + rot > q_head_dim || qo_rot0 + rot > qo_head_dim) return OXR_BAD_ARGUMENT;
+    if (rank <= 0 || down_stride < rank + rot || rot < 0 || 2 * half > rot || q_rot0 + rot > q_head_dim || qo_rot0 + rot > qo_head_dim) return OXR_BAD_ARGUMENT;
     if (dtype == 0)
-        latent_prep_kernel<float><<<n_tokens, 128, 0, stream>>>((float*)pool, slot_stride, pool_slots, (const float*)down, rank, rot, weight, eps, (const float*)q, heads,
-                                                               q_head_dim, q_rot0, (float*)q_out, qo_head_dim, qo_rot0, cos_t, sin_t, half, slots, status);
+        latent_prep_kernel<float><<<n_tokens, 128, 0, stream>>>((float*)pool, slot_stride, pool_slots, (const float*)down, down_stride, rank, rot, weight, eps, (const float*)q, heads,
+                                                               q_head_dim, q_rot0, (float*)q_out, qo_head_dim, qo_rot0, cos_t, sin_t, half, halves, slots, status);
     else
-        latent_prep_kernel<__nv_bfloat16><<<n_tokens, 128, 0, stream>>>((__nv_bfloat16*)pool, slot_stride, pool_slots, (const __nv_bfloat16*)down, rank, rot, weight,
+        latent_prep_kernel<__nv_bfloat16><<<n_tokens, 128, 0, stream>>>((__nv_bfloat16*)pool, slot_stride, pool_slots, (const __nv_bfloat16*)down, down_stride, rank, rot, weight,
                                                                        eps, (const __nv_bfloat16*)q, heads, q_head_dim, q_rot0, (__nv_bfloat16*)q_out, qo_head_dim,
-                                                                       qo_rot0, cos_t, sin_t, half, slots, status);
+                                                                       qo_rot0, cos_t, sin_t, half, halves, slots, status);
+    return oxr_launch_status();
+}
+
+// out[t] = x[t, 0:width] / rms * weight for rows `stride` apart (columns of a wider product): fp32 arithmetic, one rounding. One block per row.
+template <typename T>
+__global__ void cols_rms_norm_kernel(T* __restrict__ out, const T* __restrict__ x, int stride, int width, const float* __restrict__ weight, float eps) {
+    __shared__ float red[32];
+    const T* row = x + (size_t)blockIdx.x * stride;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = Num<T>::to_f32(row[i]);
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)blockIdx.x * width + i] = Num<T>::from_f32(Num<T>::to_f32(row[i]) * inv * weight[i]);
+}
+
+OXR_API int oxr_cols_rms_norm(void* out, const void* x, int n, int stride, int width, const float* weight, float eps, int dtype, cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (width <= 0 || stride < width) return OXR_BAD_ARGUMENT;
+    const int threads = width >= 1024 ? 256 : 128;
+    if (dtype == 0) cols_rms_norm_kernel<float><<<n, threads, 0, stream>>>((float*)out, (const float*)x, stride, width, weight, eps);
+    else cols_rms_norm_kernel<__nv_bfloat16><<<n, threads, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, stride, width, weight, eps);
     return oxr_launch_status();
 }
 

@@ -113,8 +113,9 @@ __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.lau
 inline int oxr_chain_kernels = 0;   // one per library: set through oxr_set_chain()
 
 // What the gated epilogue of a product computes from a gate sum g and an up sum u. kind 0: silu(g) * u. kind 1: with
-// g' = min(g, limit) and u' = clamp(u, -limit, limit): g' * sigmoid(alpha g') * (u' + 1). The launchers of the gated products
-// hand the library's current form to their kernels by value; oxr_set_gate_form() sets it (before each gated call).
+// g' = min(g, limit) and u' = clamp(u, -limit, limit): g' * sigmoid(alpha g') * (u' + 1). kind 3: gelu(g) * u with the tanh form of
+// gelu (kind 2 is a plain product's relu(x)^2, which has no up sum). The launchers of the gated products hand
+// the library's current form to their kernels by value; oxr_set_gate_form() sets it (before each gated call).
 struct GateForm {
     int kind;
     float alpha;
@@ -126,6 +127,10 @@ __device__ __forceinline__ float gate_apply(const GateForm& f, float g, float u)
         g = fminf(g, f.limit);
         u = fminf(fmaxf(u, -f.limit), f.limit) + 1.f;
         return __fdividef(g, 1.f + __expf(-f.alpha * g)) * u;
+    }
+    if (f.kind == 3) {   // 0.5 (1 + tanh y) is the logistic function of 2 y
+        const float y = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+        return __fdividef(g, 1.f + __expf(-2.f * y)) * u;
     }
     return __fdividef(g, 1.f + __expf(-g)) * u;   // the fast division: two ulp, far inside a bf16 step
 }

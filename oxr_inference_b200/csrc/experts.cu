@@ -6,7 +6,9 @@
 // tie); their weights are their s divided by the sum of the chosen s (+ 1e-20), times `scale`. All of it in fp32.
 // Variants, each an argument: scores that are the softmax of z over all experts instead of sigmoids (score_kind 1); a group's
 // score that is its largest s instead of the sum of its two largest (group_kind 1); weights that are the chosen s themselves,
-// times `scale`, not divided by their sum (renorm 0).
+// times `scale`, not divided by their sum (renorm 0); choice scores s + correction[e] (groups and experts are then picked by these, the
+// weights stay those of s); and identity experts: of the E scored experts the last E - real return their input, so that they need no product:
+// the token's weights for them are added up in `kept` [tokens], and the dense row has the real experts' columns only.
 //
 // For steps of many tokens the experts run one after the other instead, each over the tokens that chose it (`expert_sort`, `gather_rows`,
 // then per expert two products and the activation, then `combine_rows`): the work is then that of the chosen experts only.
@@ -21,31 +23,30 @@ constexpr int ROUTE_MAX_TOP = 32;
 constexpr int ROUTE_MAX_GROUPS = 64;
 
 __global__ void route_kernel(float* __restrict__ gate, int* __restrict__ ids, float* __restrict__ wts, const float* __restrict__ z, int n_tokens,
-                             int E, int top, int groups, int keep, float scale, int score_kind, int group_kind, int renorm) {
+                             int E, int top, int groups, int keep, float scale, int score_kind, int group_kind, int renorm, const float* __restrict__ correction,
+                             int real, float* __restrict__ kept) {
     const int t = blockIdx.x * blockDim.x + threadIdx.x;
     if (t >= n_tokens) return;
-    float* row = gate + (size_t)t * E;          // scratch for the scores until the last pass
     const float* zr = z + (size_t)t * E;
+    float zmax = -INFINITY, den = 0.f;
     if (score_kind == 1) {
-        float zmax = -INFINITY, den = 0.f;
         for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, zr[e]);
-        for (int e = 0; e < E; ++e) { row[e] = expf(zr[e] - zmax); den += row[e]; }
-        for (int e = 0; e < E; ++e) row[e] = row[e] / den;
-    } else {
-        for (int e = 0; e < E; ++e) row[e] = 1.f / (1.f + expf(-zr[e]));
+        for (int e = 0; e < E; ++e) den += expf(zr[e] - zmax);
     }
+    auto score_of = [&](int e) { return score_kind == 1 ? expf(zr[e] - zmax) / den : 1.f / (1.f + expf(-zr[e])); };
+    auto choice_of = [&](int e) { return correction != nullptr ? score_of(e) + correction[e] : score_of(e); };
     unsigned long long allowed = ~0ull;        // one bit per group
     const int per = E / groups;
     if (groups > 1 && keep < groups) {
         float score[ROUTE_MAX_GROUPS];
         for (int g = 0; g < groups; ++g) {
-            float a = -1.f, b = -1.f;           // the two largest of the group (scores are >= 0)
+            float a = -INFINITY, b = -INFINITY; // the two largest of the group
             for (int e = g * per; e < (g + 1) * per; ++e) {
-                const float v = row[e];
+                const float v = choice_of(e);
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            score[g] = group_kind == 1 ? a : a + (b >= 0.f ? b : 0.f);
+            score[g] = group_kind == 1 ? a : a + (b > -INFINITY ? b : 0.f);
         }
         allowed = 0ull;
         for (int i = 0; i < keep; ++i) {
@@ -63,21 +64,28 @@ __global__ void route_kernel(float* __restrict__ gate, int* __restrict__ ids, fl
         int best = -1;
         float best_v = -INFINITY;
         for (int e = 0; e < E; ++e) {
-            const float v = row[e];             // -1 once chosen
-            if (v >= 0.f && ((allowed >> (e / per)) & 1ull) && v > best_v) { best_v = v; best = e; }
+            bool taken = false;
+            for (int j = 0; j < i; ++j) taken |= chosen[j] == e;
+            if (taken || !((allowed >> (e / per)) & 1ull)) continue;
+            const float v = choice_of(e);
+            if (v > best_v) { best_v = v; best = e; }
         }
         chosen[i] = best;
-        chosen_s[i] = best >= 0 ? best_v : 0.f;
-        if (best >= 0) { row[best] = -1.f; sum += best_v; }
+        chosen_s[i] = best >= 0 ? score_of(best) : 0.f;
+        sum += chosen_s[i];
     }
     const float norm = renorm ? scale / (sum + 1e-20f) : scale;
-    for (int e = 0; e < E; ++e) row[e] = 0.f;
+    float* row = gate + (size_t)t * real;
+    float same = 0.f;
+    for (int e = 0; e < real; ++e) row[e] = 0.f;
     for (int i = 0; i < top; ++i) {
         const float w = chosen_s[i] * norm;
-        if (chosen[i] >= 0) row[chosen[i]] = w;
+        if (chosen[i] >= real) same += w;
+        else if (chosen[i] >= 0) row[chosen[i]] = w;
         ids[(size_t)t * top + i] = chosen[i];
         wts[(size_t)t * top + i] = w;
     }
+    if (kept != nullptr) kept[t] = same;
 }
 
 
@@ -97,12 +105,14 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 
 __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gate, int* __restrict__ ids, float* __restrict__ wts, const float* __restrict__ z,
                                                         int n_tokens, int E, int top, int groups, int keep, float scale, int score_kind,
-                                                        int group_kind, int renorm) {
-    __shared__ float sc[4][ROUTE_WARP_MAX_E];
+                                                        int group_kind, int renorm, const float* __restrict__ correction, int real,
+                                                        float* __restrict__ kept) {
+    __shared__ float sc[4][ROUTE_WARP_MAX_E], ch[4][ROUTE_WARP_MAX_E];     // scores, choice scores
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * 4 + warp;
     if (t >= n_tokens) return;
     float* s = sc[warp];
+    float* cs = ch[warp];
     const int per = E / groups;
     if (score_kind == 1) {
         float zmax = -INFINITY, den = 0.f;
@@ -114,18 +124,19 @@ __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gat
     } else {
         for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-z[(size_t)t * E + e]));
     }
+    for (int e = lane; e < E; e += 32) cs[e] = correction != nullptr ? s[e] + correction[e] : s[e];     // each lane reads what it wrote
     __syncwarp();
     unsigned allowed = 0xffffffffu;            // one bit per group
     if (groups > 1 && keep < groups) {
         float score = -INFINITY;               // lane g: group g
         if (lane < groups) {
-            float a = -1.f, b = -1.f;
+            float a = -INFINITY, b = -INFINITY;
             for (int e = lane * per; e < (lane + 1) * per; ++e) {
-                const float v = s[e];
+                const float v = cs[e];
                 if (v > a) { b = a; a = v; }
                 else if (v > b) b = v;
             }
-            score = group_kind == 1 ? a : a + (b >= 0.f ? b : 0.f);
+            score = group_kind == 1 ? a : a + (b > -INFINITY ? b : 0.f);
         }
         allowed = 0u;
         for (int i = 0; i < keep; ++i) {
@@ -141,37 +152,47 @@ __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gat
         float v = -INFINITY;
         int idx = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float x = s[e];              // -1 once chosen
-            if (x >= 0.f && ((allowed >> (e / per)) & 1u) && x > v) { v = x; idx = e; }
+            const float x = cs[e];             // -inf once chosen
+            if (((allowed >> (e / per)) & 1u) && x > v) { v = x; idx = e; }
         }
         warp_argmax(v, idx);
-        if (idx >= E) { idx = -1; v = 0.f; }       // nothing left to pick (scores that are not numbers): no expert, no weight
-        if (lane == i) { mine = idx; mine_s = v; }
-        if (lane == 0 && idx >= 0) s[idx] = -1.f;
-        sum += v;
+        if (idx >= E) idx = -1;                // nothing left to pick (scores that are not numbers): no expert, no weight
+        const float sv = idx >= 0 ? s[idx] : 0.f;
+        if (lane == i) { mine = idx; mine_s = sv; }
+        __syncwarp();
+        if (lane == 0 && idx >= 0) cs[idx] = -INFINITY;
+        sum += sv;
         __syncwarp();
     }
     const float norm = renorm ? scale / (sum + 1e-20f) : scale;
-    for (int e = lane; e < E; e += 32) gate[(size_t)t * E + e] = 0.f;
+    for (int e = lane; e < real; e += 32) gate[(size_t)t * real + e] = 0.f;
     __syncwarp();
+    const float w = lane < top ? mine_s * norm : 0.f;
     if (lane < top) {
-        const float w = mine_s * norm;
-        if (mine >= 0) gate[(size_t)t * E + mine] = w;
+        if (mine >= 0 && mine < real) gate[(size_t)t * real + mine] = w;
         ids[(size_t)t * top + lane] = mine;
         wts[(size_t)t * top + lane] = w;
+    }
+    if (kept != nullptr) {
+        float same = 0.f;                      // in the order of the picks
+        for (int i = 0; i < top; ++i) {
+            const float wi = __shfl_sync(0xffffffffu, w, i);
+            if (__shfl_sync(0xffffffffu, mine, i) >= real) same += wi;
+        }
+        if (lane == 0) kept[t] = same;
     }
 }
 
 OXR_API int oxr_route(float* gate, int* ids, float* wts, const float* z, int n_tokens, int E, int top, int groups, int keep, float scale,
-                      int score_kind, int group_kind, int renorm, cudaStream_t stream) {
+                      int score_kind, int group_kind, int renorm, const float* correction, int real, float* kept, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || top > ROUTE_MAX_TOP || groups <= 0 || groups > ROUTE_MAX_GROUPS || E % groups || keep <= 0 || keep > groups ||
+    if (real <= 0 || real > E || (real < E && kept == nullptr) || E <= 0 || top <= 0 || top > E || top > ROUTE_MAX_TOP || groups <= 0 || groups > ROUTE_MAX_GROUPS || E % groups || keep <= 0 || keep > groups ||
         top > keep * (E / groups) || score_kind < 0 || score_kind > 1 || group_kind < 0 || group_kind > 1)
         return OXR_BAD_ARGUMENT;
     if (E <= ROUTE_WARP_MAX_E && groups <= 32)
-        route_warp_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm);
+        route_warp_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept);
     else
-        route_kernel<<<(n_tokens + 63) / 64, 64, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm);
+        route_kernel<<<(n_tokens + 63) / 64, 64, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept);
     return oxr_launch_status();
 }
 
@@ -331,10 +352,11 @@ OXR_API int oxr_gather_rows(void* out, const void* x, const int* order, int rows
     return oxr_launch_status();
 }
 
-// out[t] = sum_j weights[t, j] * y[place[t top + j]], summed in fp32 in the order of j, rounded once
+// out[t] = kept[t] * x[t] + sum_j weights[t, j] * y[place[t top + j]] (x and kept: the identity experts' share, optional), summed in fp32 with the
+// sum over j in the order of j, rounded once
 template <typename T>
 __global__ void combine_rows_kernel(T* __restrict__ out, const T* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights,
-                                    int top, int width) {
+                                    int top, int width, const T* __restrict__ x, const float* __restrict__ kept) {
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float acc = 0.f;
@@ -342,16 +364,17 @@ __global__ void combine_rows_kernel(T* __restrict__ out, const T* __restrict__ y
             const int at = place[(size_t)t * top + j];
             if (at >= 0) acc = fmaf(weights[(size_t)t * top + j], Num<T>::to_f32(y[(size_t)at * width + c]), acc);
         }
+        if (x != nullptr) acc = fmaf(kept[t], Num<T>::to_f32(x[(size_t)t * width + c]), acc);
         out[(size_t)t * width + c] = Num<T>::from_f32(acc);
     }
 }
 
-OXR_API int oxr_combine_rows(void* out, const void* y, const int* place, const float* weights, int n_tokens, int top, int width, int dtype,
-                             cudaStream_t stream) {
+OXR_API int oxr_combine_rows(void* out, const void* y, const int* place, const float* weights, int n_tokens, int top, int width, const void* x, const float* kept,
+                             int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top <= 0 || width <= 0) return OXR_BAD_ARGUMENT;
-    if (dtype == 0) combine_rows_kernel<float><<<n_tokens, 256, 0, stream>>>((float*)out, (const float*)y, place, weights, top, width);
-    else combine_rows_kernel<__nv_bfloat16><<<n_tokens, 256, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)y, place, weights, top, width);
+    if (dtype == 0) combine_rows_kernel<float><<<n_tokens, 256, 0, stream>>>((float*)out, (const float*)y, place, weights, top, width, (const float*)x, kept);
+    else combine_rows_kernel<__nv_bfloat16><<<n_tokens, 256, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)y, place, weights, top, width, (const __nv_bfloat16*)x, kept);
     return oxr_launch_status();
 }
 
@@ -442,21 +465,22 @@ OXR_API int oxr_scale_placed_rows(void* x, const int* place, const float* weight
     return oxr_launch_status();
 }
 
-// y[t] += sigmoid(z[t]) * s[t]: a second feed-forward's result joins the first's, multiplied by one gate per token (z fp32 logits).
+// y[t] += g(z[t]) * s[t]: a second feed-forward's result joins the first's, multiplied by one number per token: g(z) = sigmoid(z) (z a gate's
+// fp32 logit) or z itself (`raw`).
 template <typename T>
-__global__ void add_row_gated_kernel(T* __restrict__ y, const T* __restrict__ s, const float* __restrict__ z, int hidden, size_t total) {
+__global__ void add_row_gated_kernel(T* __restrict__ y, const T* __restrict__ s, const float* __restrict__ z, int hidden, int raw, size_t total) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
-    const float g = 1.f / (1.f + expf(-z[i / hidden]));
+    const float zt = z[i / hidden], g = raw ? zt : 1.f / (1.f + expf(-zt));
     y[i] = Num<T>::from_f32(Num<T>::to_f32(y[i]) + g * Num<T>::to_f32(s[i]));
 }
 
-OXR_API int oxr_add_row_gated(void* y, const void* s, const float* z, int n, int hidden, int dtype, cudaStream_t stream) {
+OXR_API int oxr_add_row_gated(void* y, const void* s, const float* z, int n, int hidden, int raw, int dtype, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (hidden <= 0) return OXR_BAD_ARGUMENT;
     const size_t total = (size_t)n * hidden;
     const unsigned blocks = (unsigned)((total + 255) / 256);
-    if (dtype == 0) add_row_gated_kernel<float><<<blocks, 256, 0, stream>>>((float*)y, (const float*)s, z, hidden, total);
-    else add_row_gated_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)y, (const __nv_bfloat16*)s, z, hidden, total);
+    if (dtype == 0) add_row_gated_kernel<float><<<blocks, 256, 0, stream>>>((float*)y, (const float*)s, z, hidden, raw, total);
+    else add_row_gated_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((__nv_bfloat16*)y, (const __nv_bfloat16*)s, z, hidden, raw, total);
     return oxr_launch_status();
 }

@@ -8,6 +8,7 @@
 //   value  = y of the key head, when the values are the filtered keys (else the value projection, copied)
 //   norm   = y / sqrt(mean(y^2) + eps) [* weight]                   before or after the rotation
 //   rotate : (a, b) = (y_i, y_(i + half)) -> (a cos - b sin, b cos + a sin) for i < half, angles per token; the rest passes
+//   factor : a query head times a number of its own (a temperature of its scores)
 //
 // Earlier tokens of the same request are read from the step's own rows, tokens before the step from the request's tail (fp32, the last
 // n - 1 projected values of every filtered channel, the oldest first, each a row of all channels); a second kernel moves the tails on
@@ -32,6 +33,7 @@ struct PrepArgs {
     int norm_after;          // the norm comes after the rotation
     const float* q_weight;   // [DK]
     const float* k_weight;
+    const float* q_factor;   // [H]: head h's queries are multiplied by it at the end, or null
     float eps;
     const float* cos_t;      // [tokens, half] or null
     const float* sin_t;
@@ -118,6 +120,7 @@ __global__ void __launch_bounds__(128) head_prep_kernel(T* __restrict__ q_out, T
         for (int d = lane; d < a.DK; d += 32) s2 = fmaf(y[d], y[d], s2);
         inv = 1.f / sqrtf(warp_sum(s2) / (float)a.DK + a.eps);
     }
+    if (is_q && a.q_factor != nullptr) inv *= a.q_factor[h];
     T* dst = is_q ? q_out + ((size_t)t * a.H + h) * a.DK : k_pool + ((long long)slot * a.KV + h) * a.DK;
     for (int d = lane; d < a.DK; d += 32) dst[d] = Num<T>::from_f32(y[d] * inv * ((a.norm == 1 && a.norm_after) ? weight[d] : 1.f));
 }
@@ -259,6 +262,11 @@ __global__ void __launch_bounds__(128) head_prep_bf16x8_kernel(__nv_bfloat16* __
         for (int i = 0; i < 8; ++i) y[i] = y[i] * inv * wn[i];
     }
     if (live) {
+        if (is_q && a.q_factor != nullptr) {
+            const float f = a.q_factor[h];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[i] *= f;
+        }
         bf16* dst = is_q ? q_out + ((size_t)t * a.H + h) * a.DK : k_pool + ((long long)slot * a.KV + h) * a.DK;
         *reinterpret_cast<uint4*>(dst + 8 * l) = prep_pack(y);
     }
@@ -287,7 +295,7 @@ __global__ void prep_tail_kernel(const T* __restrict__ proj, const PrepArgs a, i
 
 OXR_API int oxr_head_prep(void* q_out, void* k_pool, void* v_pool, const void* proj, int n_tokens, int n_requests, int stride, int q_col0, int k_col0,
                           int v_col0, int H, int KV, int DK, int DV, int has_k, int v_mode, const float* bias, const float* taps, const float* taps_t, int n_taps, float* tails,
-                          long long tail_stride, int norm, int norm_after, const float* q_weight, const float* k_weight, float eps, const float* cos_t,
+                          long long tail_stride, int norm, int norm_after, const float* q_weight, const float* k_weight, const float* q_factor, float eps, const float* cos_t,
                           const float* sin_t, int half, const int* slots, long long pool_slots, const int* req_of_token, const int* cu_q,
                           const int* state_slots, int dtype, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
@@ -297,7 +305,7 @@ OXR_API int oxr_head_prep(void* q_out, void* k_pool, void* v_pool, const void* p
     PrepArgs a;
     a.stride = stride; a.q_col0 = q_col0; a.k_col0 = k_col0; a.v_col0 = v_col0; a.H = H; a.KV = KV; a.DK = DK; a.DV = DV; a.has_k = has_k;
     a.v_mode = has_k ? v_mode : 0; a.bias = bias; a.taps = taps; a.taps_t = taps_t; a.n_taps = taps != nullptr ? n_taps : 0; a.channels = H * DK + (has_k ? KV * DK : 0); a.tails = tails; a.tail_stride = tail_stride;
-    a.norm = norm; a.norm_after = norm_after; a.q_weight = q_weight; a.k_weight = k_weight; a.eps = eps; a.cos_t = half > 0 ? cos_t : nullptr;
+    a.norm = norm; a.norm_after = norm_after; a.q_weight = q_weight; a.k_weight = k_weight; a.q_factor = q_factor; a.eps = eps; a.cos_t = half > 0 ? cos_t : nullptr;
     a.sin_t = sin_t; a.half = half; a.slots = slots; a.pool_slots = pool_slots; a.req_of_token = req_of_token; a.cu_q = cu_q;
     a.state_slots = state_slots; a.status = status;
     const int heads = H + (has_k ? KV : 0) + (a.v_mode == 1 ? KV : 0);

@@ -193,6 +193,20 @@ __global__ void clamped_glu_bf16x8_kernel(uint4* __restrict__ out, const uint4* 
     out[row * inter8 + c] = f32_to_bf16x8(o);
 }
 
+// ---------------------------------------------------------------------------------------------- gelu-gated unit
+// out = gelu(g) * u with the tanh form gelu(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))); gate_up as in the clamped unit.
+__device__ __forceinline__ float gelu_tanh_of(float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+template <typename T>
+__global__ void gelu_glu_kernel(T* __restrict__ out, const T* __restrict__ gate_up, int inter, int interleave, size_t total) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t row = i / inter;
+        const int col = (int)(i % inter);
+        const size_t gi = interleave ? row * 2 * inter + (size_t)(col / interleave) * 2 * interleave + col % interleave : row * 2 * inter + col;
+        out[i] = Num<T>::from_f32(gelu_tanh_of(Num<T>::to_f32(gate_up[gi])) * Num<T>::to_f32(gate_up[gi + (interleave ? interleave : inter)]));
+    }
+}
+
 // ---------------------------------------------------------------------------------------------- rotary angles
 // cos/sin [tokens, half] of position * freq[i], the product and the functions in fp64, rounded once to fp32.
 __global__ void rotary_angles_kernel(float* __restrict__ cos_out, float* __restrict__ sin_out, const int* __restrict__ positions,
@@ -276,6 +290,15 @@ OXR_API int oxr_clamped_glu(void* out, const void* gate_up, int n, int inter, in
     if (dtype == 0) clamped_glu_kernel<float><<<grid_for(total, 256), 256, 0, stream_>>>((float*)out, (const float*)gate_up, inter, interleave, alpha, limit, total);
     else clamped_glu_kernel<__nv_bfloat16><<<grid_for(total, 256), 256, 0, stream_>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, inter, interleave,
                                                                                      alpha, limit, total);
+    return oxr_launch_status();
+}
+
+OXR_API int oxr_gelu_glu(void* out, const void* gate_up, int n, int inter, int interleave, int dtype, cudaStream_t stream_) {
+    if (n <= 0) return 0;
+    if (inter <= 0 || interleave < 0 || (interleave && inter % interleave)) return OXR_BAD_ARGUMENT;
+    const size_t total = (size_t)n * inter;
+    if (dtype == 0) gelu_glu_kernel<float><<<grid_for(total, 256), 256, 0, stream_>>>((float*)out, (const float*)gate_up, inter, interleave, total);
+    else gelu_glu_kernel<__nv_bfloat16><<<grid_for(total, 256), 256, 0, stream_>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, inter, interleave, total);
     return oxr_launch_status();
 }
 
@@ -648,6 +671,20 @@ OXR_API int oxr_pair_norm_mean(void* out, const void* a, const void* b, const fl
     const int threads = hidden >= 2048 ? 256 : 128;
     if (dtype == 0) pair_norm_mean_kernel<float><<<n, threads, 0, stream_>>>((float*)out, (const float*)a, (const float*)b, wa, wb, hidden, eps);
     else pair_norm_mean_kernel<__nv_bfloat16><<<n, threads, 0, stream_>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)b, wa, wb, hidden, eps);
+    return oxr_launch_status();
+}
+
+// out = fa * a + fb * b element by element (fp32, rounded once; out may be a): two mixers' results with a factor each.
+template <typename T>
+__global__ void scaled_sum_kernel(T* out, const T* a, const T* __restrict__ b, float fa, float fb, size_t total) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+        out[i] = Num<T>::from_f32(fa * Num<T>::to_f32(a[i]) + fb * Num<T>::to_f32(b[i]));
+}
+
+OXR_API int oxr_scaled_sum(void* out, const void* a, const void* b, float fa, float fb, long long total, int dtype, cudaStream_t stream_) {
+    if (total <= 0) return 0;
+    if (dtype == 0) scaled_sum_kernel<float><<<grid_for((size_t)total, 256), 256, 0, stream_>>>((float*)out, (const float*)a, (const float*)b, fa, fb, (size_t)total);
+    else scaled_sum_kernel<__nv_bfloat16><<<grid_for((size_t)total, 256), 256, 0, stream_>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)a, (const __nv_bfloat16*)b, fa, fb, (size_t)total);
     return oxr_launch_status();
 }
 

@@ -22,6 +22,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Mapping
 
+from oxr_inference_b200.config.fields import need as _need, nonneg_int as _int, pos_int as _pos_int
 from oxr_inference_b200.config.model_config import ConfigError
 from oxr_inference_b200.config.registry import Architecture, register_architecture
 from oxr_inference_b200.parts.spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
@@ -33,26 +34,6 @@ MAX_POSITIONS = 1 << 20
 """The design has no table over positions and config.json gives no limit; this bounds a request's length for the scheduler."""
 
 _SWIGLU_NAMES = {"gate_proj.weight": "gate", "up_proj.weight": "up", "down_proj.weight": "down"}
-
-
-def _need(d: Mapping[str, Any], key: str, where: str) -> Any:
-    if not isinstance(d, Mapping) or key not in d:
-        raise ConfigError(f"config.json: {where} lacks {key!r}")
-    return d[key]
-
-
-def _pos_int(d: Mapping[str, Any], key: str, where: str) -> int:
-    v = _need(d, key, where)
-    if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
-        raise ConfigError(f"config.json: {where}.{key} must be a positive integer, got {v!r}")
-    return v
-
-
-def _int(d: Mapping[str, Any], key: str, where: str) -> int:
-    v = _need(d, key, where)
-    if isinstance(v, bool) or not isinstance(v, int) or v < 0:
-        raise ConfigError(f"config.json: {where}.{key} must be an integer >= 0, got {v!r}")
-    return v
 
 
 @dataclass(frozen=True)

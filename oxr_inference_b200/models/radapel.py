@@ -15,6 +15,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Mapping
 
+from oxr_inference_b200.config.fields import need as _need, pos_int as _pos_int
 from oxr_inference_b200.config.model_config import ConfigError
 from oxr_inference_b200.config.registry import Architecture, register_architecture
 from oxr_inference_b200.parts.spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
@@ -23,19 +24,6 @@ MAX_POSITIONS = 1 << 20
 """The design has no table over positions and config.json gives no limit; this bounds a request's length for the scheduler."""
 GATE_ALPHA = 1.702
 """Slope of the sigmoid that stands in for GELU in the feed-forward's gate; fixed by the design."""
-
-
-def _need(d: Mapping[str, Any], key: str, where: str) -> Any:
-    if not isinstance(d, Mapping) or key not in d:
-        raise ConfigError(f"config.json: {where} lacks {key!r}")
-    return d[key]
-
-
-def _pos_int(d: Mapping[str, Any], key: str, where: str) -> int:
-    v = _need(d, key, where)
-    if isinstance(v, bool) or not isinstance(v, int) or v <= 0:
-        raise ConfigError(f"config.json: {where}.{key} must be a positive integer, got {v!r}")
-    return v
 
 
 @dataclass(frozen=True)

@@ -68,6 +68,14 @@ _raw_stream = getattr(torch._C, "_cuda_getCurrentRawStream", None)
 _raw_device = getattr(torch._C, "_cuda_getDevice", None) or torch.cuda.current_device
 
 
+def _need_rows(t: torch.Tensor, name: str, dtype: torch.dtype | None = None) -> None:
+    """Like :func:`_need` for a matrix whose rows may lie apart (columns of a wider one); the entries of a row lie side by side."""
+    if not t.is_cuda:
+        raise KernelError(f"{name} is on {t.device}; the kernels run on a CUDA device only (there is no CPU path)")
+    if t.dim() != 2 or t.stride(1) != 1 or t.stride(0) < t.shape[1] or (dtype is not None and t.dtype != dtype):
+        raise KernelError(f"{name}: {t.dtype} {tuple(t.shape)} with strides {t.stride()} is not rows of {dtype or 'one dtype'}")
+
+
 def _stream() -> int:
     """Handle of the current CUDA stream. The raw getter costs a fraction of a microsecond; `torch.cuda.current_stream()`
     builds a Stream object per call (several microseconds, per kernel launch of an eager step)."""
@@ -136,19 +144,20 @@ def _lib():
         lib.oxr_gated_group_norm.argtypes = [p, p, p, i, i, i, p, i, i, f, i, p]
         lib.oxr_attention_rows.argtypes = [p, p, i, p, ll, i, p, ll, i, i, i, i, i, i, p, p, p, i, i, i, f, i, i, i, p, i, p, i, p, p]
         lib.oxr_scatter_rows.argtypes = [p, ll, ll, p, i, i, i, p, i, i, p, p, ll, i, p]
-        lib.oxr_latent_prep.argtypes = [p, ll, ll, p, i, i, p, f, p, i, i, i, p, i, i, p, p, i, p, i, i, p, p]
+        lib.oxr_latent_prep.argtypes = [p, ll, ll, p, i, i, i, p, f, p, i, i, i, p, i, i, p, p, i, i, p, i, i, p, p]
+        lib.oxr_cols_rms_norm.argtypes = [p, p, i, i, i, p, f, i, p]
         lib.oxr_head_linear.argtypes = [p, i, i, p, i, i, p, i, i, i, i, i, p]
         lib.oxr_conv_qkv_store.argtypes = [p, p, p, i, i, i, i, i, i, i, p, p, p, p, ll, p, p, p, p, f, i, p, p, p, p, p, ll, i, i, i, i, i, i, i, p, p]
         lib.oxr_add_bias.argtypes = [p, p, i, i, i, p]
         lib.oxr_scale_f32.argtypes = [p, f, ll, p]
         lib.oxr_mlstm_scan.argtypes = [p, p, p, i, i, i, i, i, p, p, i, i, i, f, f, p, ll, p, p, i, p]
         lib.oxr_head_norm_gate.argtypes = [p, p, p, i, i, i, p, i, i, f, i, i, p]
-        lib.oxr_route.argtypes = [p, p, p, p, i, i, i, i, i, f, i, i, i, p]
+        lib.oxr_route.argtypes = [p, p, p, p, i, i, i, i, i, f, i, i, i, p, i, p, p]
         lib.oxr_gated_relu2.argtypes = [p, p, p, i, i, i, i, p]
         lib.oxr_expert_sort.argtypes = [p, p, p, p, p, i, i, i, i, p]
         lib.oxr_gemm_tcgen05_grouped_bf16.argtypes = [p, p, p, i, i, i, i, p, i, i, i, p, p]
         lib.oxr_gather_rows.argtypes = [p, p, p, i, i, i, i, p]
-        lib.oxr_combine_rows.argtypes = [p, p, p, p, i, i, i, i, p]
+        lib.oxr_combine_rows.argtypes = [p, p, p, p, i, i, i, p, p, i, p]
         lib.oxr_stream_layer_norm.argtypes = [p, p, p, p, p, i, i, f, i, p]
         lib.oxr_gated_residual.argtypes = [p, p, p, p, p, p, i, p, p, i, p, i, i, i, p]
         lib.oxr_gated_residual_norm.argtypes = [p, p, p, p, p, p, p, i, p, p, i, p, i, i, p, p, f, i, p]
@@ -162,16 +171,24 @@ def _lib():
         lib.oxr_attention_mix_mma_smem.argtypes = [i, i, i, i, i, i]
         lib.oxr_attention_mix_mma_smem.restype = c_longlong
         lib.oxr_expert_clamped_glu.argtypes = [p, p, p, i, i, i, f, f, i, p]
-        lib.oxr_head_prep.argtypes = [p, p, p, p, i, i, i, i, i, i, i, i, i, i, i, i, p, p, p, i, p, ll, i, i, p, p, f, p, p, i, p, ll, p, p, p, i, p, p]
+        lib.oxr_head_prep.argtypes = [p, p, p, p, i, i, i, i, i, i, i, i, i, i, i, i, p, p, p, i, p, ll, i, i, p, p, p, f, p, p, i, p, ll, p, p, p, i, p, p]
         lib.oxr_sigmoid_gate.argtypes = [p, p, i, i, i, i, i, i, i, p]
         lib.oxr_gla_scan.argtypes = [p, p, i, i, i, i, i, p, p, f, i, i, i, f, p, ll, p, p, i, i, p]
         lib.oxr_pair_norm_mean.argtypes = [p, p, p, p, p, i, i, f, i, p]
         lib.oxr_tanh_cap.argtypes = [p, f, ll, p]
         lib.oxr_expert_silu_glu.argtypes = [p, p, p, i, i, i, i, i, p]
         lib.oxr_scale_placed_rows.argtypes = [p, p, p, i, i, i, p]
-        lib.oxr_add_row_gated.argtypes = [p, p, p, i, i, i, p]
+        lib.oxr_add_row_gated.argtypes = [p, p, p, i, i, i, i, p]
+        lib.oxr_gelu_glu.argtypes = [p, p, i, i, i, i, p]
+        lib.oxr_scaled_sum.argtypes = [p, p, p, f, f, ll, i, p]
+        lib.oxr_shift_norm.argtypes = [p, p, p, p, p, f, p, f, p, p, ll, p, p, p, i, i, i, i, p]
+        lib.oxr_delta_scan.argtypes = [p, p, i, i, i, i, i, p, i, p, p, i, p, f, f, i, i, i, p, ll, p, p, i, i, p]
+        lib.oxr_tanh_cols.argtypes = [p, p, i, i, i, i, i, p]
+        lib.oxr_diff_prep.argtypes = [p, p, p, p, i, i, i, i, i, i, i, i, i, i, i, p, p, ll, i, p, p]
+        lib.oxr_diff_combine.argtypes = [p, p, i, i, i, i, p, f, f, i, p]
         for name in ("oxr_head_prep", "oxr_sigmoid_gate", "oxr_gla_scan", "oxr_pair_norm_mean", "oxr_tanh_cap", "oxr_expert_silu_glu",
-                     "oxr_scale_placed_rows", "oxr_add_row_gated"):
+                     "oxr_scale_placed_rows", "oxr_add_row_gated", "oxr_cols_rms_norm", "oxr_gelu_glu", "oxr_scaled_sum", "oxr_shift_norm",
+                     "oxr_delta_scan", "oxr_tanh_cols", "oxr_diff_prep", "oxr_diff_combine"):
             getattr(lib, name).restype = c_int
         for name in ("oxr_stream_layer_norm", "oxr_gated_residual", "oxr_gelu_tanh", "oxr_attention_mix_rows", "oxr_bias_rope_store", "oxr_gated_residual_norm",
                      "oxr_expert_clamped_glu"):
@@ -343,14 +360,14 @@ def gated_silu_linear(x: torch.Tensor, weight: torch.Tensor, interleave: int = 0
     return gated_linear(x, weight, interleave)
 
 
-GATE_KINDS = {"silu": 0, "clamped": 1}
+GATE_KINDS = {"silu": 0, "clamped": 1, "gelu": 3}
 
 
 def gated_linear(x: torch.Tensor, weight: torch.Tensor, interleave: int = 0, *, kind: str = "silu", alpha: float = 1.0,
                  limit: float = 0.0) -> torch.Tensor:
     """``gate_form(x Wg^T, x Wu^T)`` for a weight that stacks Wg and Wu: side by side (``interleave`` 0: one product,
     then the activation kernel) or alternating in groups of 8 rows. ``kind`` "silu": ``silu(g) * u``; "clamped": with ``g' = min(g, limit)``
-    and ``u' = clamp(u, -limit, limit)``, ``g' * sigmoid(alpha g') * (u' + 1)``. With alternating rows a bf16 product runs the kernel
+    and ``u' = clamp(u, -limit, limit)``, ``g' * sigmoid(alpha g') * (u' + 1)``; "gelu": ``gelu(g) * u`` with the tanh form of gelu. With alternating rows a bf16 product runs the kernel
     ``linear`` would pick for its size (skinny, one-SM or two-SM tcgen05) with an epilogue that applies the form to the fp32
     sums and writes the gated product alone; 32-bit runs the product and then the activation kernel on interleaved columns.
     ``x`` may be a :class:`NormedLazily`."""
@@ -384,6 +401,8 @@ def gated_linear(x: torch.Tensor, weight: torch.Tensor, interleave: int = 0, *, 
         return out
     if kind == "silu":
         return silu_mul(linear(x, weight), interleave)
+    if kind == "gelu":
+        return gelu_glu(linear(x, weight), interleave)
     return clamped_glu(linear(x, weight), alpha=alpha, limit=limit, interleave=interleave)
 
 
@@ -1127,6 +1146,18 @@ def clamped_glu(gate_up: torch.Tensor, *, alpha: float, limit: float, interleave
     return out
 
 
+def gelu_glu(gate_up: torch.Tensor, interleave: int = 0) -> torch.Tensor:
+    """``gelu(gate) * up`` (the tanh form of gelu) for ``gate_up = [gate | up]`` along the last axis, or alternating in groups of ``interleave``
+    columns."""
+    _need(gate_up, "gate_up")
+    n, two_i = gate_up.shape
+    if two_i % 2:
+        raise KernelError("gate_up must have an even number of columns")
+    out = torch.empty((n, two_i // 2), dtype=gate_up.dtype, device=gate_up.device)
+    _done(_lib().oxr_gelu_glu(out.data_ptr(), gate_up.data_ptr(), n, two_i // 2, int(interleave), _dtype_code(gate_up), _stream()), "gelu_glu")
+    return out
+
+
 def rotary_angles(positions: torch.Tensor, freq: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
     """fp32 ``cos`` and ``sin`` ``[tokens, len(freq)]`` of ``position * freq[i]`` for this step's tokens; the product and the functions are
     evaluated in fp64 (``freq`` is a float64 device tensor) and rounded once, so the table is exact to fp32 at any position."""
@@ -1433,21 +1464,35 @@ def scatter_rows(pool: torch.Tensor, src: torch.Tensor, col0: int, slots: torch.
 
 def latent_prep(pool: torch.Tensor, down: torch.Tensor, rank: int, rot: int, weight: torch.Tensor, eps: float, q: torch.Tensor, heads: int,
                 q_head_dim: int, q_rot0: int, q_out: torch.Tensor, qo_head_dim: int, qo_rot0: int, cos: torch.Tensor, sin: torch.Tensor,
-                slots: torch.Tensor, status: torch.Tensor) -> None:
+                slots: torch.Tensor, status: torch.Tensor, halves: bool = False) -> None:
     """Per token: the latent cache row ``[rmsnorm(down[:rank]) * weight | rotate(down[rank:])]`` goes to ``pool[slot]`` (slot -1: not stored), and
-    every head's rotated query part ``rotate(q[h, q_rot0 : q_rot0 + rot])`` to ``q_out[h, qo_rot0 : ...]``. ``rotate`` turns entry pairs (2i, 2i+1)
-    by the token's angle i (``cos``/``sin`` ``[tokens, half]``); entries past ``2 * half`` pass unchanged."""
+    every head's rotated query part ``rotate(q[h, q_rot0 : q_rot0 + rot])`` to ``q_out[h, qo_rot0 : ...]``. ``rotate`` turns entry pairs (2i, 2i+1),
+    or with ``halves`` the pairs (i, i + half), by the token's angle i (``cos``/``sin`` ``[tokens, half]``); entries past ``2 * half`` pass
+    unchanged. ``down`` may be columns of a wider product (rows apart, entries of a row side by side)."""
     _need(pool, "pool")
-    _need(down, "down", pool.dtype)
+    _need_rows(down, "down", pool.dtype)
     _need(q, "q", pool.dtype)
     _need(q_out, "q_out", pool.dtype)
     _need(cos, "cos", torch.float32)
     n = down.shape[0]
     if down.shape[1] != rank + rot or pool[0, 0].numel() != rank + rot:
         raise KernelError("latent_prep: sizes of the down projection and the pool do not fit")
-    _done(_lib().oxr_latent_prep(pool.data_ptr(), rank + rot, pool.shape[0] * pool.shape[1], down.data_ptr(), rank, rot, weight.data_ptr(), float(eps),
+    _done(_lib().oxr_latent_prep(pool.data_ptr(), rank + rot, pool.shape[0] * pool.shape[1], down.data_ptr(), down.stride(0), rank, rot, weight.data_ptr(), float(eps),
                                  q.data_ptr(), heads, q_head_dim, q_rot0, q_out.data_ptr(), qo_head_dim, qo_rot0, cos.data_ptr(), sin.data_ptr(),
-                                 cos.shape[1], slots.data_ptr(), n, _dtype_code(down), status.data_ptr(), _stream()), "latent_prep")
+                                 cos.shape[1], int(bool(halves)), slots.data_ptr(), n, _dtype_code(down), status.data_ptr(), _stream()), "latent_prep")
+
+
+def cols_rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """``x / sqrt(mean(x^2) + eps) * weight`` row by row (fp32 arithmetic, one rounding) for columns of a wider product."""
+    _need_rows(x, "x")
+    _need(weight, "weight", torch.float32)
+    n, width = x.shape
+    if weight.numel() != width:
+        raise KernelError("cols_rms_norm: one weight per column")
+    out = torch.empty((n, width), dtype=x.dtype, device=x.device)
+    _done(_lib().oxr_cols_rms_norm(out.data_ptr(), x.data_ptr(), n, x.stride(0), width, weight.data_ptr(), float(eps), _dtype_code(x), _stream()),
+          "cols_rms_norm")
+    return out
 
 
 def head_linear(out: torch.Tensor, out0: int, x: torch.Tensor, x0: int, weight: torch.Tensor) -> torch.Tensor:
@@ -1635,19 +1680,33 @@ ROUTE_GROUP_SCORES = {"top2_sum": 0, "max": 1}
 
 
 def route(z: torch.Tensor, *, top: int, groups: int, keep: int, scale: float, score: str = "sigmoid", group_score: str = "top2_sum",
-          renormalize: bool = True) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+          renormalize: bool = True, correction: torch.Tensor | None = None,
+          kept: torch.Tensor | None = None, identity: int = 0) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
     """Router logits ``z [tokens, E]`` (fp32) to the choice of ``top`` experts per token. Scores are ``sigmoid(z)`` or, with ``score="softmax"``,
     the softmax of z over all experts; of ``groups`` equal groups of neighbouring experts only the ``keep`` best may be chosen from, a group's
     score being the sum of its two best scores (``"top2_sum"``) or its best score (``"max"``); the weights are the chosen scores over their sum
-    (``renormalize``) or as they are, times ``scale``. Returns ``gate [tokens, E]`` (fp32: a chosen expert's weight, else 0), ``ids [tokens, top]``
-    (int32) and ``weights [tokens, top]`` (fp32)."""
+    (``renormalize``) or as they are, times ``scale``. With ``correction [E]`` (fp32) groups and experts are chosen by score + correction; the weights
+    stay those of the scores. The last ``identity`` of the E experts return their input: the sum of a token's weights for them goes to ``kept
+    [tokens]`` (fp32). Returns ``gate [tokens, E - identity]`` (fp32: a chosen expert's weight, else 0), ``ids [tokens, top]`` (int32) and ``weights
+    [tokens, top]`` (fp32)."""
     _need(z, "z", torch.float32)
     n, E = z.shape
-    gate = torch.empty((n, E), dtype=torch.float32, device=z.device)
+    if not 0 <= identity < E:
+        raise KernelError(f"route: {identity} identity experts of {E}")
+    if correction is not None:
+        _need(correction, "correction", torch.float32)
+        if correction.numel() != E:
+            raise KernelError("route: one correction per expert")
+    gate = torch.empty((n, E - identity), dtype=torch.float32, device=z.device)
+    if identity:
+        _need(kept, "kept", torch.float32)
+        if kept.numel() != n:
+            raise KernelError("route: kept holds one number per token")
     ids = torch.empty((n, top), dtype=torch.int32, device=z.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=z.device)
     _done(_lib().oxr_route(gate.data_ptr(), ids.data_ptr(), wts.data_ptr(), z.data_ptr(), n, E, int(top), int(groups), int(keep), float(scale),
-                           ROUTE_SCORES[score], ROUTE_GROUP_SCORES[group_score], int(bool(renormalize)), _stream()), "route")
+                           ROUTE_SCORES[score], ROUTE_GROUP_SCORES[group_score], int(bool(renormalize)), _ptr(correction), E - identity,
+                           _ptr(kept) if identity else None, _stream()), "route")
     return gate, ids, wts
 
 
@@ -1743,17 +1802,25 @@ def gather_rows(x: torch.Tensor, order: torch.Tensor, per_row: int) -> torch.Ten
     return out
 
 
-def combine_rows(y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor) -> torch.Tensor:
-    """``out[t] = sum_j weights[t, j] * y[place[t * top + j]]`` with the sum in fp32 in the order of j; ``y [>= tokens * top, width]``."""
+def combine_rows(y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, x: torch.Tensor | None = None, kept: torch.Tensor | None = None) -> torch.Tensor:
+    """``out[t] = sum_j weights[t, j] * y[place[t * top + j]]`` with the sum in fp32 in the order of j; ``y [>= tokens * top, width]``. With ``x [tokens,
+    width]`` and ``kept [tokens]`` (fp32) ``kept[t] * x[t]`` is added: the share of experts that return their input."""
     _need(y, "y")
     _need(place, "place", torch.int32)
     _need(weights, "weights", torch.float32)
     n, top = weights.shape
     if place.numel() != n * top or y.shape[0] < n * top:
         raise KernelError("combine_rows: sizes do not fit")
+    if (x is None) != (kept is None):
+        raise KernelError("combine_rows: the kept input comes with its weights or not at all")
+    if x is not None:
+        _need(x, "x", y.dtype)
+        _need(kept, "kept", torch.float32)
+        if x.shape != (n, y.shape[1]) or kept.numel() != n:
+            raise KernelError("combine_rows: sizes do not fit")
     out = torch.empty((n, y.shape[1]), dtype=y.dtype, device=y.device)
-    _done(_lib().oxr_combine_rows(out.data_ptr(), y.data_ptr(), place.data_ptr(), weights.data_ptr(), n, top, y.shape[1], _dtype_code(y), _stream()),
-          "combine_rows")
+    _done(_lib().oxr_combine_rows(out.data_ptr(), y.data_ptr(), place.data_ptr(), weights.data_ptr(), n, top, y.shape[1], _ptr(x), _ptr(kept), _dtype_code(y),
+                                  _stream()), "combine_rows")
     return out
 
 
@@ -1764,7 +1831,7 @@ HEAD_NORMS = {None: 0, "weighted": 1, "unit": 2}
 def head_prep(proj: torch.Tensor, *, q_col0: int, k_col0: int | None, v_col0: int | None, values_are_keys: bool = False, num_heads: int,
               num_kv_heads: int, key_dim: int, value_dim: int, bias: torch.Tensor | None = None, taps: torch.Tensor | None = None,
               taps_t: torch.Tensor | None = None, tails: torch.Tensor | None = None, norm: str | None = None, norm_after_rotation: bool = False, q_weight: torch.Tensor | None = None,
-              k_weight: torch.Tensor | None = None, eps: float = 0.0, cos: torch.Tensor | None = None, sin: torch.Tensor | None = None,
+              k_weight: torch.Tensor | None = None, q_factor: torch.Tensor | None = None, eps: float = 0.0, cos: torch.Tensor | None = None, sin: torch.Tensor | None = None,
               k_pool: torch.Tensor | None = None, v_pool: torch.Tensor | None = None, slots: torch.Tensor, req_of_token: torch.Tensor,
               cu_q: torch.Tensor, state_slots: torch.Tensor, n_requests: int, status: torch.Tensor) -> torch.Tensor:
     """Query and key heads on their way from the projections ``proj [tokens, *]`` to attention, and the cache write. In this order, each step
@@ -1772,7 +1839,8 @@ def head_prep(proj: torch.Tensor, *, q_col0: int, k_col0: int | None, v_col0: in
     the current token; ``taps_t``, the same transposed, lets the 16-byte bfloat16 kernel run; earlier tokens come from the step's rows or from
     the request's row of ``tails``, fp32 ``[slots, (n - 1) * channels]``, the oldest value of all channels first, which is moved on afterwards); with ``values_are_keys`` the filtered keys are stored as the values; every head is RMS-normed
     (``norm="weighted"``: times ``q_weight`` / ``k_weight [DK]``; ``"unit"``: no weight) before or after the rotation; the pairs
-    ``(i, i + half)`` of each head's first ``2 half`` entries turn by the token's angles (``cos``, ``sin`` fp32 ``[tokens, half]``). Keys and
+    ``(i, i + half)`` of each head's first ``2 half`` entries turn by the token's angles (``cos``, ``sin`` fp32 ``[tokens, half]``); query head h is
+    multiplied by ``q_factor[h]`` (fp32). Keys and
     values go to ``k_pool`` / ``v_pool [pages, page_size, KV, D]`` at ``slots`` (-1: not stored); ``k_col0`` None: queries only. Returns
     ``q [tokens, H * DK]``. All arithmetic fp32, one rounding."""
     _need(proj, "proj")
@@ -1817,11 +1885,15 @@ def head_prep(proj: torch.Tensor, *, q_col0: int, k_col0: int | None, v_col0: in
     for w in (q_weight, k_weight):
         if w is not None:
             _need(w, "norm weight", torch.float32)
+    if q_factor is not None:
+        _need(q_factor, "q_factor", torch.float32)
+        if q_factor.numel() != H:
+            raise KernelError("head_prep: one factor per query head")
     q = torch.empty((n, H * DK), dtype=proj.dtype, device=proj.device)
     _done(_lib().oxr_head_prep(q.data_ptr(), _ptr(k_pool) if has_k else None, _ptr(v_pool) if has_k else None, proj.data_ptr(), n, int(n_requests),
                                proj.shape[1], int(q_col0), int(k_col0 or 0), int(v_col0 or 0), H, KV, DK, DV, int(has_k), v_mode, _ptr(bias), _ptr(taps),
                                _ptr(taps_t) if taps is not None else None, n_taps, _ptr(tails) if n_taps > 1 else None, tail_stride, HEAD_NORMS[norm], int(bool(norm_after_rotation)), _ptr(q_weight),
-                               _ptr(k_weight), float(eps), _ptr(cos), _ptr(sin), half, slots.data_ptr(), pool_slots, req_of_token.data_ptr(),
+                               _ptr(k_weight), _ptr(q_factor), float(eps), _ptr(cos), _ptr(sin), half, slots.data_ptr(), pool_slots, req_of_token.data_ptr(),
                                cu_q.data_ptr(), state_slots.data_ptr(), _dtype_code(proj), status.data_ptr(), _stream()), "head_prep")
     global launch_count
     launch_count += 1 if n_taps > 1 else 0      # the kernel that moves the tails on
@@ -1921,12 +1993,136 @@ def scale_placed_rows_(x: torch.Tensor, place: torch.Tensor, weights: torch.Tens
     return x
 
 
-def add_row_gated_(y: torch.Tensor, s: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
-    """In place ``y[t] += sigmoid(z[t]) * s[t]`` with one fp32 logit ``z[t]`` per row."""
+def add_row_gated_(y: torch.Tensor, s: torch.Tensor, z: torch.Tensor, raw: bool = False) -> torch.Tensor:
+    """In place ``y[t] += sigmoid(z[t]) * s[t]`` with one fp32 logit ``z[t]`` per row; ``raw``: ``y[t] += z[t] * s[t]``."""
     _need(y, "y")
     _need(s, "s", y.dtype)
     _need(z, "z", torch.float32)
     if s.shape != y.shape or z.numel() != y.shape[0]:
         raise KernelError("add_row_gated: sizes do not fit")
-    _done(_lib().oxr_add_row_gated(y.data_ptr(), s.data_ptr(), z.data_ptr(), y.shape[0], y.shape[1], _dtype_code(y), _stream()), "add_row_gated")
+    _done(_lib().oxr_add_row_gated(y.data_ptr(), s.data_ptr(), z.data_ptr(), y.shape[0], y.shape[1], int(bool(raw)), _dtype_code(y), _stream()), "add_row_gated")
     return y
+
+
+def scaled_sum(a: torch.Tensor, b: torch.Tensor, fa: float, fb: float) -> torch.Tensor:
+    """``fa * a + fb * b`` element by element (fp32, rounded once), written over ``a``."""
+    _need(a, "a")
+    _need(b, "b", a.dtype)
+    if a.shape != b.shape:
+        raise KernelError("scaled_sum: shapes differ")
+    _done(_lib().oxr_scaled_sum(a.data_ptr(), a.data_ptr(), b.data_ptr(), float(fa), float(fb), a.numel(), _dtype_code(a), _stream()), "scaled_sum")
+    return a
+
+
+# --------------------------------------------------------------------------------------------------- token shift
+def shift_norm(stream: torch.Tensor, weight: torch.Tensor, eps: float, shift: torch.Tensor, state: torch.Tensor, out_dtype: torch.dtype, *,
+               req_of_token: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, y: torch.Tensor | None = None,
+               post_weight: torch.Tensor | None = None, post_eps: float = 0.0, rows_per_block: int = 0) -> tuple[torch.Tensor, torch.Tensor]:
+    """``h = rmsnorm(stream) * weight`` blended with the token before: ``out_t = h_t + (h_(t-1) - h_t) * shift`` (``shift [hidden]`` fp32), rounded to
+    ``out_dtype``. ``h_(t-1)`` of a request's first token in the step comes from its row of ``state`` (fp32 ``[slots, hidden]``, rows may lie
+    apart), which moves on to the request's last token. With ``y`` the stream first becomes ``stream + rmsnorm(y) * post_weight`` (in a new
+    tensor): an add that the layer before left to do. Returns ``(out, stream)``. ``rows_per_block``: neighbouring tokens per block of threads
+    (0: chosen by the step's size)."""
+    _need(stream, "stream", torch.float32)
+    _need(weight, "weight", torch.float32)
+    _need(shift, "shift", torch.float32)
+    n, hidden = stream.shape
+    if state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[1] != hidden:
+        raise KernelError("shift_norm: the state must be fp32 rows of the stream's width")
+    if weight.numel() != hidden or shift.numel() != hidden:
+        raise KernelError("shift_norm: one weight and one share per entry")
+    new = stream
+    if y is not None:
+        _need(y, "y", out_dtype)
+        _need(post_weight, "post_weight", torch.float32)
+        if y.shape != stream.shape:
+            raise KernelError(f"shift_norm: y {tuple(y.shape)} does not match the stream {tuple(stream.shape)}")
+        new = torch.empty_like(stream)
+    out = torch.empty((n, hidden), dtype=out_dtype, device=stream.device)
+    rows = rows_per_block or (1 if n <= 2 * num_sms() else 4)
+    _done(_lib().oxr_shift_norm(out.data_ptr(), stream.data_ptr(), _ptr(y), new.data_ptr() if y is not None else None, _ptr(post_weight), float(post_eps),
+                                weight.data_ptr(), float(eps), shift.data_ptr(), state.data_ptr(), state.stride(0), req_of_token.data_ptr(), cu_q.data_ptr(),
+                                state_slots.data_ptr(), n, hidden, int(rows), _DT[out_dtype], _stream()), "shift_norm")
+    return out, new
+
+
+# --------------------------------------------------------------------------------------------------- delta rule
+def tanh_cols(z: torch.Tensor, col0: int, width: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """``tanh(z[:, col0 : col0 + width])`` of an fp32 product, rounded to ``out_dtype``."""
+    _need(z, "z", torch.float32)
+    out = torch.empty((z.shape[0], width), dtype=out_dtype, device=z.device)
+    _done(_lib().oxr_tanh_cols(out.data_ptr(), z.data_ptr(), z.shape[0], z.shape[1], int(col0), int(width), _DT[out_dtype], _stream()), "tanh_cols")
+    return out
+
+
+def delta_scan(proj: torch.Tensor, r_col0: int, k_col0: int, v_col0: int, zw: torch.Tensor, w_bias: torch.Tensor, za: torch.Tensor, a_bias: torch.Tensor, *,
+               heads: int, key_dim: int, value_dim: int, rate: float, len_eps: float, state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
+               n_requests: int, columns_per_thread: int = 0) -> torch.Tensor:
+    """The delta rule with a decay per key channel over a packed step: per head, with ``u = k / sqrt(sum k^2 + len_eps)``, ``w = exp(-rate *
+    sigmoid(zw + w_bias))`` and ``a = sigmoid(za + a_bias)``,
+
+        S_t = diag(w) S_(t-1) - (a * u) (u^T S_(t-1)) + k v^T        o_t = S_t^T r
+
+    ``proj`` holds r, k and v head by head from the given columns; ``zw`` and ``za`` (fp32 ``[tokens, >= heads * key_dim]``, the first columns) are the
+    logits of decay and removal rate; ``state`` (fp32, first axis the slot: S transposed, ``[heads, value_dim, key_dim]``) is read and left at the
+    state after each request's last token. Returns fp32 ``o [tokens, heads * value_dim]``. ``columns_per_thread`` (1 or 2) forces the kernel's
+    split; 0 chooses by the step's shape."""
+    _need(proj, "proj")
+    _need(zw, "zw", torch.float32)
+    _need(za, "za", torch.float32)
+    _need(w_bias, "w_bias", torch.float32)
+    _need(a_bias, "a_bias", torch.float32)
+    keys = heads * key_dim
+    if state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[1] < keys * value_dim:
+        raise KernelError("delta_scan: the state must be fp32 rows of heads x value_dim x key_dim")
+    n = proj.shape[0]
+    if zw.shape[0] != n or za.shape[0] != n or zw.shape[1] < keys or za.shape[1] < keys or w_bias.numel() != keys or a_bias.numel() != keys:
+        raise KernelError("delta_scan: decay and rate logits must be [tokens, heads * key_dim] with one bias each")
+    if max(r_col0 + keys, k_col0 + keys, v_col0 + heads * value_dim) > proj.shape[1]:
+        raise KernelError("delta_scan: the columns of r, k and v do not fit the projections")
+    y = torch.empty((n, heads * value_dim), dtype=torch.float32, device=proj.device)
+    _done(_lib().oxr_delta_scan(y.data_ptr(), proj.data_ptr(), int(n_requests), proj.shape[1], int(r_col0), int(k_col0), int(v_col0), zw.data_ptr(),
+                                zw.shape[1], w_bias.data_ptr(), za.data_ptr(), za.shape[1], a_bias.data_ptr(), float(rate), float(len_eps), int(heads),
+                                int(key_dim), int(value_dim), state.data_ptr(), state.stride(0), cu_q.data_ptr(), state_slots.data_ptr(),
+                                _dtype_code(proj), int(columns_per_thread or 1), _stream()), "delta_scan")
+    return y
+
+
+# --------------------------------------------------------------------------------------------------- differential attention
+def diff_prep(proj: torch.Tensor, *, num_heads: int, num_kv_heads: int, dim: int, value_dim: int, width: int, bias: torch.Tensor | None,
+              k_pool: torch.Tensor, v_pool: torch.Tensor, slots: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
+    """Query, key and value heads of differential attention on their way from ``proj [tokens, 2 H D + 2 G D + G DV]`` (+ ``bias``, fp32) to an attention
+    kernel. Returns ``q [tokens, 2 H * width]``: query head 2h + m holds map m of head h at its place ``m D`` of a row of ``width >= 2 D`` entries and
+    zeros elsewhere, so that over key rows ``[k1 | k2]`` (``k_pool [pages, page_size, G, width]``) it scores ``q_m . k_m``. Keys and values go to their
+    slots (-1: not stored); ``v_pool [pages, page_size, G, >= DV]``. Entries of the pools behind 2 D and DV are not written."""
+    _need(proj, "proj")
+    _need(k_pool, "k_pool", proj.dtype)
+    _need(v_pool, "v_pool", proj.dtype)
+    n, cols = proj.shape
+    H, G, D, DV = int(num_heads), int(num_kv_heads), int(dim), int(value_dim)
+    need = 2 * H * D + 2 * G * D + G * DV
+    if cols != need or tuple(k_pool.shape[2:]) != (G, width) or v_pool.shape[2] != G or v_pool.shape[:2] != k_pool.shape[:2]:
+        raise KernelError("diff_prep: the projections or the pools do not fit the heads")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != need:
+            raise KernelError("diff_prep: one bias per projected column")
+    q = torch.empty((n, 2 * H * width), dtype=proj.dtype, device=proj.device)
+    _done(_lib().oxr_diff_prep(q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), proj.data_ptr(), n, cols, 0, 2 * H * D, 2 * (H + G) * D, H, G, D, DV,
+                               int(width), v_pool.shape[3], _ptr(bias), slots.data_ptr(), k_pool.shape[0] * k_pool.shape[1], _dtype_code(proj),
+                               status.data_ptr(), _stream()), "diff_prep")
+    return q
+
+
+def diff_combine(o: torch.Tensor, num_heads: int, value_dim: int, lam: torch.Tensor, eps: float, factor: float) -> torch.Tensor:
+    """Per head ``o1 - lam * o2`` of the two maps' outputs (``o [tokens, 2 H, >= value_dim]``, ``lam`` one fp32 number on the device), over its root mean
+    square, times ``factor``: ``[tokens, H * value_dim]``."""
+    _need(o, "o")
+    _need(lam, "lam", torch.float32)
+    n, heads, width = o.shape
+    if heads != 2 * num_heads or width < value_dim or lam.numel() != 1:
+        raise KernelError("diff_combine: sizes do not fit")
+    out = torch.empty((n, num_heads * value_dim), dtype=o.dtype, device=o.device)
+    _done(_lib().oxr_diff_combine(out.data_ptr(), o.data_ptr(), n, width, int(num_heads), int(value_dim), lam.data_ptr(), float(eps), float(factor),
+                                  _dtype_code(o), _stream()), "diff_combine")
+    return out

@@ -1,6 +1,6 @@
 """Parts a decoder is assembled from; importing the package registers the built-in ones."""
 
-from oxr_inference_b200.parts import (attention, block, experts, gated_attention, gla, joint, masked_attention, mamba, mlp, mlstm, norm,  # noqa: F401
+from oxr_inference_b200.parts import (attention, block, delta, differential, experts, gated_attention, gla, joint, masked_attention, mamba, mlp, mlstm, norm,  # noqa: F401
                                       paired, rope)  # noqa: F401  (register themselves)
 from oxr_inference_b200.parts.base import (ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, JOINTS, MIXERS, NORMS, POSITION_ENCODINGS,
                                            DeferredLinear, Embedding, FeedForward, GroupView, Head, Joint, LayerCache, Mixer, Norm, PagedKVNeed,

@@ -5,7 +5,8 @@ from __future__ import annotations
 import torch
 
 from oxr_inference_b200 import ops
-from oxr_inference_b200.parts.base import ARRANGEMENTS, DeferredLinear, FeedForward, LayerCache, Mixer, Norm, ParamInfo, Part, Runtime, StepContext
+from oxr_inference_b200.parts.base import (ARRANGEMENTS, DeferredLinear, FeedForward, LayerCache, Mixer, Norm, ParamInfo, Part, Runtime, StateNeed,
+                                           StepContext)
 from oxr_inference_b200.parts.linear import StackedLinear
 
 
@@ -110,6 +111,84 @@ class SandwichNormBlock:
         h = self.mixer_post_norm.add_normed(stream, a, then=self.feed_forward_norm)
         self.feed_forward_post_norm.add_normed(stream, self.feed_forward.forward(h))
         return None, stream
+
+
+@ARRANGEMENTS.register("shifted_sandwich_norm")
+class ShiftedSandwichNormBlock(SandwichNormBlock, Part):
+    """``sandwich_norm`` with a token shift in front of the mixer: with ``h = pre_norm(x)`` the mixer reads ``h + (h' - h) * shift`` entry by entry, where
+    ``h'`` is the previous token's h (zeros before the first token) and ``shift [hidden]`` a tensor of the block. The last token's h is part of a
+    request's state: ``cache_need`` is the mixer's with one fp32 row appended to its state.
+
+    A block may leave the add of its last sublayer to the next block of this kind (:class:`PendingNormedAdd`), whose first kernel then does
+    both: post-norm, add, pre-norm and shift are one pass over the rows."""
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, feed_forward: FeedForward | None, feed_forward_norm: Norm | None, *, runtime: Runtime,
+                 hidden_size: int, mixer_post_norm: Norm, feed_forward_post_norm: Norm | None = None):
+        super().__init__(mixer, mixer_norm, feed_forward, feed_forward_norm, mixer_post_norm=mixer_post_norm,
+                         feed_forward_post_norm=feed_forward_post_norm)
+        for norm in (mixer_norm, mixer_post_norm, feed_forward_post_norm):
+            if norm is not None and not hasattr(norm, "shifted"):
+                raise ValueError("the shifted_sandwich_norm arrangement is built for norms that offer the shifted form (rms_norm)")
+        from oxr_inference_b200.cache.plan import split_need   # here: the cache package imports the parts' interfaces
+
+        self.runtime, self.hidden = runtime, int(hidden_size)
+        self.shift: torch.Tensor | None = None
+        self._paged, self._mixer_state = split_need(mixer.cache_need())
+        if self._mixer_state is not None and (self._mixer_state.dtype != torch.float32 or len(self._mixer_state.shape) != 1):
+            raise ValueError("the mixer's state must be an fp32 row to share one with the shift's")
+        self._mixer_cols = self._mixer_state.shape[0] if self._mixer_state is not None else 0
+        self._shift_col = (self._mixer_cols + 3) // 4 * 4      # rows of whole 16-byte words
+
+    def parameters(self) -> dict[str, ParamInfo]:
+        return {"shift": ParamInfo((self.hidden,), role="vector")}
+
+    def assign(self, name: str, tensor: torch.Tensor) -> None:
+        if name != "shift":
+            raise KeyError(name)
+        self.shift = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
+
+    def cache_need(self):
+        state = StateNeed(((self._shift_col + self.hidden + 3) // 4 * 4,), torch.float32)
+        return state if self._paged is None else (self._paged, state)
+
+    def keeps_add_for(self, after) -> bool:
+        """Whether ``after`` (the block that runs next, or None) takes this block's last add into its first norm."""
+        return isinstance(after, ShiftedSandwichNormBlock)
+
+    def forward(self, x, residual: torch.Tensor | None, ctx: StepContext, cache: LayerCache, defer_output: bool = False):
+        pending = None
+        if isinstance(x, PendingNormedAdd):
+            pending, stream = x, residual
+        elif residual is None:
+            if isinstance(x, DeferredLinear):
+                x = x.materialize()
+            if x.dtype != torch.float32:
+                raise ValueError("this arrangement keeps the stream in fp32: the embedding must hand it over whole")
+            stream = x
+        elif x is not None:
+            raise ValueError("this arrangement takes the stream whole; the block before it left an output that is not yet added")
+        else:
+            stream = residual
+        shift_state = cache.state[:, self._shift_col:self._shift_col + self.hidden]
+        h, stream = self.mixer_norm.shifted(stream, self.shift, shift_state, ctx, pending)
+        mixer_state = cache.state[:, :self._mixer_cols] if self._mixer_cols else None     # a view: the kernels take the row stride
+        a = self.mixer.forward(h, ctx, LayerCache(group=cache.group, layer_in_group=cache.layer_in_group, store=cache.store, state=mixer_state))
+        if self.feed_forward is None:
+            last = PendingNormedAdd(a, self.mixer_post_norm)
+        else:
+            h = self.mixer_post_norm.add_normed(stream, a, then=self.feed_forward_norm)
+            last = PendingNormedAdd(self.feed_forward.forward(h), self.feed_forward_post_norm)
+        if defer_output:
+            return last, stream
+        last.norm.add_normed(stream, last.y)
+        return None, stream
+
+
+class PendingNormedAdd:
+    """A sublayer's result whose post-norm and add into the stream are still to do: ``stream += norm(y)``."""
+
+    def __init__(self, y: torch.Tensor, norm: Norm):
+        self.y, self.norm = y, norm
 
 
 @ARRANGEMENTS.register("output_norm")

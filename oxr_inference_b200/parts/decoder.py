@@ -118,10 +118,16 @@ class DecoderModel:
                 raise ValueError(f"schedule entry {i} names joint {entry.joint}; the model has {len(self.joints)}")
         self.schedule = spec.schedule
         self.cache_plan: CachePlan = make_cache_plan(
-            [self.blocks[e.layer].mixer.cache_need() for e in self.schedule], [e.cache_of for e in self.schedule])
+            [self._cache_need(self.blocks[e.layer]) for e in self.schedule], [e.cache_of for e in self.schedule])
         self.tile_specs = sorted({spec for b in self.blocks for spec in b.mixer.tile_specs()})
 
     # ---- construction helpers
+    @staticmethod
+    def _cache_need(block):
+        """What one run of a block keeps: its mixer's need, unless the arrangement keeps something of its own beside it."""
+        own = getattr(block, "cache_need", None)
+        return own() if own is not None else block.mixer.cache_need()
+
     def _position(self, spec: PartSpec | None):
         if spec is None:
             return None

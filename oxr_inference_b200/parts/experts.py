@@ -18,7 +18,9 @@ class RoutedExperts(FeedForward):
     ``s = sigmoid(z)`` or the softmax of z over all experts (``score``). The experts form ``groups`` equal groups of neighbours; a group's
     score is the sum of its two largest scores or its largest one (``group_score``), and only experts of the ``keep`` best groups can be
     chosen. Each token runs the ``top`` allowed experts with the largest scores; their outputs are added with weights
-    ``s / (sum of the chosen s + 1e-20) * scale`` or, with ``renormalize=False``, ``s * scale``. With ``weight_on="input"`` the weight multiplies
+    ``s / (sum of the chosen s + 1e-20) * scale`` or, with ``renormalize=False``, ``s * scale``. ``choice_correction``: a learned number per expert
+    (tensor ``correction``) is added to the scores for the choice (of groups and experts) and nowhere else. ``identity``: that many more experts
+    behind the others are scored and chosen like them but have no tensors and return their input. With ``weight_on="input"`` the weight multiplies
     what the expert READS instead of what it returns: the layer's output is the sum of ``expert_i(w_i h)``. ``shared``: a feed-forward
     (``{"kind": ..., "params": {...}}``, tensors under ``shared.``) that every token runs and whose output is added; with ``shared_gate`` it is
     first multiplied by ``sigmoid(W_sg h)``, one number per token (tensor ``shared.sg [1, hidden]``, the logit in fp32).
@@ -39,7 +41,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, runtime: Runtime, *, hidden_size: int, intermediate_size: int, experts: int, top: int, groups: int = 1, keep: int = 1,
                  scale: float = 1.0, grouped_min_rows: int | None = None, activation: str = "relu2", limit: float = 0.0, alpha: float = 1.702,
                  score: str = "sigmoid", group_score: str = "top2_sum", renormalize: bool = True, shared: Mapping[str, Any] | None = None,
-                 weight_on: str = "output", shared_gate: bool = False):
+                 weight_on: str = "output", shared_gate: bool = False, choice_correction: bool = False, identity: int = 0):
         self.runtime = runtime
         if activation not in ("relu2", "clamped_glu", "silu_glu"):
             raise ValueError(f"expert activation {activation!r} is not one of 'relu2', 'clamped_glu', 'silu_glu'")
@@ -47,6 +49,8 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"weight_on {weight_on!r} is not one of 'output', 'input'")
         if weight_on == "input" and activation != "silu_glu":
             raise ValueError("weights on the experts' input are built for the SiLU-gated unit")
+        if identity < 0 or (identity and weight_on == "input"):
+            raise ValueError("identity experts need weights on the output, and a number of at least 0")
         if shared_gate and not shared:
             raise ValueError("a gate on the shared expert needs a shared expert")
         self.activation, self.on_input, self.shared_gate = activation, weight_on == "input", bool(shared_gate)
@@ -59,21 +63,25 @@ class RoutedExperts(FeedForward):
         self.shared = FEED_FORWARDS.build(shared["kind"], runtime, **shared.get("params", {})) if shared else None
         self.hidden, self.ff, self.E, self.top = int(hidden_size), int(intermediate_size), int(experts), int(top)
         self.groups, self.keep, self.scale = int(groups), int(keep), float(scale)
-        if self.groups < 1 or self.E % self.groups:
-            raise ValueError(f"{self.E} experts do not form {self.groups} equal groups")
+        self.identity, self.scored = int(identity), int(experts) + int(identity)
+        self.has_correction, self.correction = bool(choice_correction), None
+        if self.groups < 1 or self.scored % self.groups:
+            raise ValueError(f"{self.scored} experts do not form {self.groups} equal groups")
         if not 1 <= self.keep <= self.groups:
             raise ValueError(f"{self.keep} of {self.groups} groups cannot be kept")
-        if not 1 <= self.top <= self.keep * (self.E // self.groups):
-            raise ValueError(f"{self.top} experts cannot be chosen from {self.keep} groups of {self.E // self.groups}")
+        if not 1 <= self.top <= self.keep * (self.scored // self.groups):
+            raise ValueError(f"{self.top} experts cannot be chosen from {self.keep} groups of {self.scored // self.groups}")
         self.grouped_min_rows = self.GROUPED_MIN_ROWS if grouped_min_rows is None else int(grouped_min_rows)
         self.up_rows = (2 if self.gated else 1) * self.ff     # rows of one expert in the stack: [gate | up] for a gated unit
         self.up: torch.Tensor | None = None       # [E * up_rows, hidden]
         self.down: torch.Tensor | None = None     # [hidden, E * ff]
         self.down_by_expert: torch.Tensor | None = None   # [E, hidden, ff]: made at the first grouped step
-        self.router: torch.Tensor | None = None   # [E, hidden]
+        self.router: torch.Tensor | None = None   # [E + identity, hidden]
 
     def parameters(self) -> dict[str, ParamInfo]:
-        out = {"router": ParamInfo((self.E, self.hidden))}
+        out = {"router": ParamInfo((self.scored, self.hidden))}
+        if self.has_correction:
+            out["correction"] = ParamInfo((self.scored,), role="vector")
         for e in range(self.E):
             if self.gated:
                 out[f"e{e}.gate"] = ParamInfo((self.ff, self.hidden))
@@ -105,6 +113,9 @@ class RoutedExperts(FeedForward):
         if name == "router":
             self.router = tensor.to(device=self.runtime.device, dtype=dtype).contiguous()
             return
+        if name == "correction" and self.has_correction:
+            self.correction = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
+            return
         expert, which = name.split(".")
         e = int(expert[1:])
         if which in ("up", "gate"):
@@ -129,20 +140,25 @@ class RoutedExperts(FeedForward):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         z = ops.linear(h, self.router, torch.float32)
+        kept = torch.empty((h.shape[0],), dtype=torch.float32, device=h.device) if self.identity else None
         gate, ids, weights = ops.route(z, top=self.top, groups=self.groups, keep=self.keep, scale=self.scale, score=self.score,
-                                       group_score=self.group_score, renormalize=self.renormalize)
-        if self.top < self.E and h.shape[0] >= self.grouped_min_rows > 0 and not torch.cuda.is_current_stream_capturing():
-            y = self._grouped(h, ids, weights)
+                                       group_score=self.group_score, renormalize=self.renormalize, correction=self.correction, kept=kept,
+                                       identity=self.identity)
+        if self.top < self.scored and h.shape[0] >= self.grouped_min_rows > 0 and not torch.cuda.is_current_stream_capturing():
+            y = self._grouped(h, ids, weights, kept)
         else:
             y = ops.linear(self._act(ops.linear(h, self.up), gate), self.down)
+            if kept is not None:
+                ops.add_row_gated_(y, h, kept, raw=True)
         if self.shared is None:
             return y
         if self.shared_gate:
             return ops.add_row_gated_(y, self.shared.forward(h), ops.linear(h, self.shared_gate_weight, torch.float32))
         return ops.add_(y, self.shared.forward(h))
 
-    def _grouped(self, h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor) -> torch.Tensor:
-        """Every expert over the rows that chose it."""
+    def _grouped(self, h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, kept: torch.Tensor | None = None) -> torch.Tensor:
+        """Every expert over the rows that chose it (choices of identity experts have no place in the ordered list)."""
+        same = h if kept is not None else None
         if self.down_by_expert is None:
             # a second copy of the down-projections, expert by expert (the stacked one is laid out for the single product)
             self.down_by_expert = self.down.view(self.hidden, self.E, self.ff).permute(1, 0, 2).contiguous()
@@ -161,7 +177,7 @@ class RoutedExperts(FeedForward):
             else:
                 a = ops.grouped_linear(x, self.up, tile_group, self.ff, relu2=True)     # the activation in the product's epilogue
             y = ops.grouped_linear(a, self.down_by_expert.view(self.E * self.hidden, self.ff), tile_group, self.hidden)
-            return ops.combine_rows(y, place, weights)
+            return ops.combine_rows(y, place, weights, same, kept)
         counts, order, place, _ = ops.expert_sort(ids, self.E)
         x = ops.gather_rows(h, order, self.top)                  # [tokens * top, hidden], ordered by expert
         if self.on_input:
@@ -174,4 +190,4 @@ class RoutedExperts(FeedForward):
                 u = ops.linear(x[at:at + c], self.up[e * self.up_rows:(e + 1) * self.up_rows])
                 ops.linear(self._act(u, None), self.down_by_expert[e], out=y[at:at + c])
                 at += c
-        return ops.combine_rows(y, place, weights)
+        return ops.combine_rows(y, place, weights, same, kept)

@@ -22,6 +22,7 @@ class GatedAttention(Mixer):
     * ``values_are_keys``: there is no value projection; the values are the keys as they leave the filter (before norm and rotation).
     * ``qk_norm``: ``"weighted"`` = per-head RMS norm times ``q.norm`` / ``k.norm [key_dim]`` (shared by the heads), ``"unit"`` = without a weight;
       ``norm_after_rotation`` puts it behind the rotation instead of before it.
+    * ``head_temperature``: the scores of head h are multiplied by a learned number (tensor ``temp [heads]``).
     * a position encoding with per-step angles (``step_angles``) turns the pairs ``(i, i + half)`` of each q and k head.
     * mask: causal; ``window`` > 0: position i sees j only if ``i - j < window`` or ``j < keep_first``.
     * ``sink``: a learned number per head (tensor ``sink``) whose exponential joins the softmax denominator; no key, no value, not scaled.
@@ -37,7 +38,8 @@ class GatedAttention(Mixer):
     def __init__(self, runtime: Runtime, position: PositionEncoding | None, *, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int,
                  value_dim: int, scale: float, eps: float = 0.0, qk_norm: str | None = None, norm_after_rotation: bool = False, qk_biases: bool = False,
                  conv_taps: int = 0, values_are_keys: bool = False, window: int = 0, keep_first: int = 0, sink: bool = False,
-                 output_gate: str | None = None, borrows_kv: bool = False, cache_window: int | None = None, cache_keep_first: int | None = None):
+                 output_gate: str | None = None, borrows_kv: bool = False, cache_window: int | None = None, cache_keep_first: int | None = None,
+                 head_temperature: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are not a multiple of {num_kv_heads} KV heads")
         if qk_norm not in ops.HEAD_NORMS:
@@ -59,7 +61,7 @@ class GatedAttention(Mixer):
         self.scale, self.eps, self.qk_norm, self.norm_after = float(scale), float(eps), qk_norm, bool(norm_after_rotation)
         self.qk_biases, self.taps, self.values_are_keys = bool(qk_biases), int(conv_taps), bool(values_are_keys)
         self.window, self.keep_first, self.has_sink, self.output_gate = int(window), int(keep_first), bool(sink), output_gate
-        self.borrows = bool(borrows_kv)
+        self.borrows, self.has_temp = bool(borrows_kv), bool(head_temperature)
         self.cache_window = self.window if cache_window is None else int(cache_window)
         self.cache_keep_first = self.keep_first if cache_keep_first is None else int(cache_keep_first)
         self.cq, self.ck = self.H * self.DK, 0 if self.borrows else self.KV * self.DK
@@ -91,6 +93,8 @@ class GatedAttention(Mixer):
             out.update({f"{n}.norm": (self.DK,) for n in sides})
         if self.has_sink:
             out["sink"] = (self.H,)
+        if self.has_temp:
+            out["temp"] = (self.H,)
         return out
 
     def parameters(self) -> dict[str, ParamInfo]:
@@ -159,7 +163,7 @@ class GatedAttention(Mixer):
         q = ops.head_prep(proj, q_col0=0, k_col0=self.cq if self.ck else None, v_col0=self.cq + self.ck if self.cv else None,
                           values_are_keys=self.values_are_keys, num_heads=self.H, num_kv_heads=self.KV, key_dim=self.DK, value_dim=self.DV,
                           bias=self.bias, taps=self.conv, taps_t=self.conv_t, tails=cache.state, norm=self.qk_norm, norm_after_rotation=self.norm_after,
-                          q_weight=v.get("q.norm"), k_weight=v.get("k.norm"), eps=self.eps, cos=cos, sin=sin, k_pool=k_pool, v_pool=v_pool,
+                          q_weight=v.get("q.norm"), k_weight=v.get("k.norm"), q_factor=v.get("temp"), eps=self.eps, cos=cos, sin=sin, k_pool=k_pool, v_pool=v_pool,
                           slots=group.slots if cache.store else ctx.no_store_slots, req_of_token=ctx.req_of_token, cu_q=ctx.cu_q,
                           state_slots=ctx.state_slots, n_requests=ctx.n_requests, status=ctx.status)
         sink = v.get("sink")

@@ -224,20 +224,26 @@ class LatentAttention(Mixer):
     the latent ``c`` and ``rot_dim`` more that are rotated into a key part shared by all heads; only ``[c | rotated part]`` is
     cached. Per head the unrotated key is ``W_uk c`` and the value ``W_uv c``; the query ``W_q h`` is laid out head by head as
     ``[key_dim unrotated | rot_dim rotated]``; the score is ``(q_u . k_u + q_r . k_r) * scale``; causal; optional ``sink``: a learned
-    number per head whose exponential joins the softmax denominator (it has no key, no value and is not scaled).
+    number per head whose exponential joins the softmax denominator (it has no key, no value and is not scaled). ``q_rank`` > 0: the query
+    passes a latent of its own, ``W_uq rmsnorm(W_dq h)`` with the weight ``dq.norm`` (tensors ``dq``, ``dq.norm``, ``uq`` in place of ``q``). Which entries
+    of the rotated part form a pair is the position encoding's (neighbours, or an entry and the one half the rotated part further on).
 
     Computed in the absorbed form, which never builds per-head keys or values: ``q_u . (W_uk c) = (W_uk^T q_u) . c``, so every head
     attends with the query ``[W_uk^T q_u | q_r]`` over the one cached row per token (whose first ``rank`` entries are the value as
     well), and ``W_uv`` is applied to the attention's output."""
 
     def __init__(self, runtime: Runtime, position: PositionEncoding | None, *, hidden_size: int, num_heads: int, key_dim: int, rot_dim: int,
-                 value_dim: int, rank: int, scale: float, eps: float, sink: bool = True):
+                 value_dim: int, rank: int, scale: float, eps: float, sink: bool = True, q_rank: int = 0):
         if rot_dim and position is None:
             raise ValueError("latent_attention with a rotated part needs a position encoding")
         self.runtime, self.position = runtime, position
         self.hidden, self.H, self.D, self.R, self.DV, self.L = int(hidden_size), int(num_heads), int(key_dim), int(rot_dim), int(value_dim), int(rank)
         self.scale, self.eps, self.has_sink = float(scale), float(eps), bool(sink)
-        self.q_dkv = StackedLinear(runtime, self.hidden, {"q": self.H * (self.D + self.R), "dkv": self.L + self.R})
+        self.QL, q_cols = int(q_rank), self.H * (self.D + self.R)
+        # everything that reads h is one product
+        self.q_dkv = StackedLinear(runtime, self.hidden, {**({"dq": self.QL} if self.QL else {"q": q_cols}), "dkv": self.L + self.R})
+        self.uq = StackedLinear(runtime, self.QL, {"uq": q_cols}) if self.QL else None
+        self.q_norm: torch.Tensor | None = None
         self.out = StackedLinear(runtime, self.H * self.DV, {"o": self.hidden})
         self.c_norm: torch.Tensor | None = None
         self.sink: torch.Tensor | None = None
@@ -250,10 +256,19 @@ class LatentAttention(Mixer):
                "uk": ParamInfo((self.H * self.D, self.L)), "uv": ParamInfo((self.H * self.DV, self.L))}
         if self.has_sink:
             out["sink"] = ParamInfo((self.H,), role="vector")
+        if self.QL:
+            out.update(self.uq.parameters())
+            out["dq.norm"] = ParamInfo((self.QL,), init="around_one", role="vector")
         return out
 
     def assign(self, name: str, tensor: torch.Tensor) -> None:
         rt = self.runtime
+        if self.QL and name == "uq":
+            self.uq.assign(name, tensor)
+            return
+        if self.QL and name == "dq.norm":
+            self.q_norm = tensor.to(device=rt.device, dtype=torch.float32).contiguous()
+            return
         if name in self.q_dkv.outs:
             self.q_dkv.assign(name, tensor)
         elif name in self.out.outs:
@@ -291,16 +306,20 @@ class LatentAttention(Mixer):
         both = self.q_dkv(h)
         if both.dtype != pool.dtype:
             both = ops.cast(both, pool.dtype)
-        q_cols = H * (D + R)
-        q = both[:, :q_cols].contiguous().view(n, H, D + R)
-        down = both[:, q_cols:].contiguous()
+        if self.QL:
+            q = self.uq(ops.cols_rms_norm(both[:, :self.QL], self.q_norm, self.eps)).view(n, H, D + R)
+            down = both[:, self.QL:]
+        else:
+            q_cols = H * (D + R)
+            q = both[:, :q_cols].contiguous().view(n, H, D + R)
+            down = both[:, q_cols:]
         if self.position is not None:
             cos, sin = self.position.step_angles(ctx)
         else:   # no rotated part at all
             cos = sin = torch.empty((n, 0), dtype=torch.float32, device=pool.device)
         q_abs = torch.empty((n, H, L + R), dtype=pool.dtype, device=pool.device)
         ops.latent_prep(pool, down, L, R, self.c_norm, self.eps, q, H, D + R, D, q_abs, L + R, L, cos, sin,
-                        group.slots if cache.store else ctx.no_store_slots, ctx.status)
+                        group.slots if cache.store else ctx.no_store_slots, ctx.status, halves=getattr(self.position, "halves", False))
         ops.head_linear(q_abs, 0, q, 0, self.uk)
         if self.tiled and pool.dtype == torch.bfloat16:
             o_lat = ops.paged_attention(q_abs, pool, pool, tiles=ctx.tiles, cu_q=ctx.cu_q, ctx_lens=ctx.ctx_lens, block_table=group.block_table,

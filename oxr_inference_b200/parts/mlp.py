@@ -1,4 +1,4 @@
-"""Dense feed-forwards: SiLU-gated, clamped gated, and a plain two-matrix layer with the tanh form of GELU."""
+"""Dense feed-forwards: SiLU-gated, clamped gated, GELU-gated, and a plain two-matrix layer with the tanh form of GELU."""
 
 from __future__ import annotations
 
@@ -70,6 +70,32 @@ class ClampedGLU(FeedForward):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         return self.down(ops.gated_linear(h, self.gate_up.weight, self.gate_up.interleave, kind="clamped", alpha=self.alpha, limit=self.limit))
+
+
+@FEED_FORWARDS.register("gelu_glu")
+class GeluGLU(FeedForward):
+    """``down( gelu_tanh(h W_gate^T) * (h W_up^T) )`` with the tanh form of GELU. Gate and up are one product whose epilogue applies the
+    activation (bfloat16, sizes that allow it)."""
+
+    def __init__(self, runtime: Runtime, *, hidden_size: int, intermediate_size: int):
+        self.hidden, self.inter = int(hidden_size), int(intermediate_size)
+        # rows alternate in groups of 8 where the size allows, as in SwiGLU: the products' epilogues then apply the gate form
+        self.gate_up = StackedLinear(runtime, self.hidden, {"gate": self.inter, "up": self.inter}, interleave=ops.GATE_UP_INTERLEAVE)
+        self.down = StackedLinear(runtime, self.inter, {"down": self.hidden})
+
+    def parameters(self) -> dict[str, ParamInfo]:
+        return {**self.gate_up.parameters(), **self.down.parameters()}
+
+    def assign(self, name: str, tensor: torch.Tensor) -> None:
+        if name in self.gate_up.outs:
+            self.gate_up.assign(name, tensor)
+        elif name in self.down.outs:
+            self.down.assign(name, tensor)
+        else:
+            raise KeyError(name)
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        return self.down(ops.gated_linear(h, self.gate_up.weight, self.gate_up.interleave, kind="gelu"))
 
 
 @FEED_FORWARDS.register("gelu_mlp")

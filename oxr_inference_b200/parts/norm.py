@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from oxr_inference_b200 import ops
-from oxr_inference_b200.parts.base import NORMS, DeferredLinear, Norm, ParamInfo, Runtime
+from oxr_inference_b200.parts.base import NORMS, DeferredLinear, Norm, ParamInfo, Runtime, StepContext
 
 
 @NORMS.register("rms_norm")
@@ -60,6 +60,16 @@ class RMSNorm(Norm):
         if then is None:
             return ops.norm_add_norm(stream, y, self.weight, self.eps, rounded=rounded)
         return ops.norm_add_norm(stream, y, self.weight, self.eps, then.weight, then.eps)
+
+
+    def shifted(self, stream: torch.Tensor, shift: torch.Tensor, state: torch.Tensor, ctx: StepContext, pending=None) -> tuple[torch.Tensor, torch.Tensor]:
+        """``h = rmsnorm(stream) * weight`` blended with the token before, ``h + (h' - h) * shift``, in the activation dtype; ``state`` holds h' of each
+        request's first token in the step and is moved on. ``pending`` (an RMS-normed add that the block before left: ``y`` and ``norm``) is added to
+        the stream in the same pass. Returns (the blended h, the stream)."""
+        dtype = self.runtime.dtype
+        post = {} if pending is None else {"y": ops.cast(pending.y, dtype), "post_weight": pending.norm.weight, "post_eps": pending.norm.eps}
+        return ops.shift_norm(stream, self.weight, self.eps, shift, state, dtype, req_of_token=ctx.req_of_token, cu_q=ctx.cu_q,
+                              state_slots=ctx.state_slots, **post)
 
 
 @NORMS.register("layer_norm")

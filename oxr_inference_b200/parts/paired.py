@@ -1,4 +1,4 @@
-"""Two mixers side by side that read the same input; what comes out is the mean of their normed results."""
+"""Two mixers side by side that read the same input; what comes out is the mean of their normed results, or a weighted sum of them."""
 
 from __future__ import annotations
 
@@ -14,16 +14,18 @@ from oxr_inference_b200.parts.base import MIXERS, POSITION_ENCODINGS, LayerCache
 class MixerPair(Mixer):
     """``0.5 * (rmsnorm(left(h)) * left.out + rmsnorm(right(h)) * right.out)``: two registered mixers (``left`` and ``right``: ``{"kind": ...,
     "params": {...}, "position": {"kind": ..., "params": {...}} or None}``, tensors under ``left.`` / ``right.``), each result RMS-normed over the
-    model width with a weight of its own before the two are averaged.
+    model width with a weight of its own before the two are averaged. With ``scales`` = (fl, fr) there is no such norm: the result is
+    ``fl * left(h) + fr * right(h)``.
 
     What the two keep between steps is kept side by side: at most one of them may keep pages of keys and values (it gets the layer's page
     group); their fixed-size states share one fp32 row per request, the left one's first."""
 
     def __init__(self, runtime: Runtime, position: PositionEncoding | None, *, hidden_size: int, eps: float, left: Mapping[str, Any],
-                 right: Mapping[str, Any]):
+                 right: Mapping[str, Any], scales: tuple[float, float] | None = None):
         if position is not None:
             raise ValueError("mixer_pair takes no position encoding of its own: each side names its own")
         self.runtime, self.hidden, self.eps = runtime, int(hidden_size), float(eps)
+        self.scales = (float(scales[0]), float(scales[1])) if scales is not None else None
         self.sides: dict[str, Mixer] = {}
         for name, spec in (("left", left), ("right", right)):
             pos = spec.get("position")
@@ -48,7 +50,7 @@ class MixerPair(Mixer):
         self.state_size = at
 
     def parameters(self) -> dict[str, ParamInfo]:
-        out = {f"{name}.out": ParamInfo((self.hidden,), init="around_one", role="vector") for name in self.sides}
+        out = {} if self.scales is not None else {f"{name}.out": ParamInfo((self.hidden,), init="around_one", role="vector") for name in self.sides}
         for name, m in self.sides.items():
             out.update({f"{name}.{local}": info for local, info in m.parameters().items()})
         return out
@@ -57,7 +59,7 @@ class MixerPair(Mixer):
         side, _, local = name.partition(".")
         if side not in self.sides or not local:
             raise KeyError(name)
-        if local == "out":
+        if local == "out" and self.scales is None:
             self.weights[side] = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
         else:
             self.sides[side].assign(local, tensor)
@@ -90,4 +92,6 @@ class MixerPair(Mixer):
         b = self.sides["right"].forward(h, ctx, self._side_cache("right", cache))
         if b.dtype != a.dtype:
             b = ops.cast(b, a.dtype)
+        if self.scales is not None:
+            return ops.scaled_sum(a, b, *self.scales)
         return ops.pair_norm_mean(a, b, self.weights["left"], self.weights["right"], self.eps)

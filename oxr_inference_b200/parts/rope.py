@@ -99,6 +99,9 @@ class RotaryHalves(PositionEncoding):
     table over positions: each step computes cos and sin ``[tokens, dims / 2]`` for its own tokens once (frequencies, product and functions in
     fp64, rounded once to fp32) and layers with equal parameters share them."""
 
+    halves = True
+    """Pairs are (i, i + dims / 2), not neighbours."""
+
     def __init__(self, runtime: Runtime, *, dims: int, base: float, scaling: dict | None = None):
         if dims % 2 or dims <= 0:
             raise ValueError(f"rotary dimension {dims} must be even and positive")
