@@ -1027,6 +1027,249 @@ def nidudra_workload(args) -> int:
     return 0
 
 
+def verorax_config(width: int, ff: int, heads: int, kv_heads: int, head_dim: int, layers: int, vocab: int, experts: int = 16, top: int = 4) -> dict:
+    """A Verorax model of a real model's layer sizes. Its layers take turns of four: latent attention (rows of 192 + 64 entries, queries through a
+    latent of a quarter of the width); differential attention over the last 1,024 keys, two maps of half a head each over whole-head values;
+    the pair (attention over the last 1,024 keys with half of each head rotated, beside the delta rule with ``width / 128`` heads of 128);
+    latent attention again. All with the head sizes of the Qwen3 model beside it. The feed-forwards alternate between a gated layer of that
+    model's size and experts (``top`` of ``experts`` and 4 identity experts, each an eighth of ``ff`` wide)."""
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top)}, "router": {"experts": experts, "identity": 4, "top": top}}
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": 64, "rot": {"dims": 64, "base": 10000.0}, "vdim": head_dim, "kv_rank": 192, "q_rank": width // 4,
+              "scale": (head_dim + 64) ** -0.5}
+    diff = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim // 2, "vdim": head_dim, "diff": 0.4, "scale": (head_dim // 2) ** -0.5, "mask": {"size": 1024}}
+    pair = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "mask": {"size": 1024},
+                     "rot": {"dims": head_dim // 2, "base": 100000.0}},
+            "right": {"heads": max(width // 128, 1), "dim": 128, "rank": 64}, "left_scale": 0.7, "right_scale": 0.6}
+    turn = (("latent_attention", latent), ("attention", diff), ("parallel", pair), ("latent_attention", latent))
+    return {"architecture": "Verorax", "norm": {"eps": 1e-6}, "vocab": vocab, "width": width,
+            "layers": [{"type": turn[i % 4][0], "mixer": turn[i % 4][1], "mlp": (dense, moe)[i % 2]} for i in range(layers)]}
+
+
+def verorax_kernels(width: int, heads: int, kv_heads: int, head_dim: int, ff: int) -> list[dict]:
+    """Each kernel of the design alone, at one model size, beside the like kernel of the paths that were there before: device time (median, L2
+    flushed between calls), the bytes or FLOPs it has to move or do, and the fraction of the measured peak."""
+    import torch
+
+    from oxr_inference_b200 import ops
+
+    dev = "cuda"
+    hbm_gbs, bf16_tflops, _ = peaks()
+    flush = torch.zeros(128 << 20, dtype=torch.float32, device=dev)
+    status = ops.new_status(dev)
+    bf = torch.bfloat16
+    rows = []
+
+    def put(name, like, fn, *, bytes_=None, flops=None):
+        ms = _time_ms(fn, flush=flush)
+        row = {"kernel": name, "like": like, "us": round(ms * 1e3, 1)}
+        if bytes_ is not None:
+            row.update(gb_s=round(bytes_ / (ms * 1e-3) / 1e9, 1), frac=round(bytes_ / (ms * 1e-3) / 1e9 / hbm_gbs, 4), bound="hbm")
+        else:
+            row.update(tflop_s=round(flops / (ms * 1e-3) / 1e12, 2), frac=round(flops / (ms * 1e-3) / 1e12 / bf16_tflops, 4), bound="tensor")
+        rows.append(row)
+
+    P, T, B, CTX = 16, 2048, 8, 2048
+    H, KV, D, L, R = heads, kv_heads, head_dim, 192, 64
+    QL, WINDOW = width // 4, 1024
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rand(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(*shape, generator=g, device=dev) * scale).to(dtype)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    n_pages = B * (CTX // P) + T // P + 8
+    k_pool, v_pool, latent_pool = rand(n_pages, P, KV, D), rand(n_pages, P, KV, D), rand(n_pages, P, 1, L + R)
+    cq, ck, cv = H * D, KV * D, KV * D
+    ones = torch.ones(D, device=dev)
+    cos_table = torch.ones(8192, D // 2, device=dev)
+    maps = ops.make_kv_maps(k_pool.unsqueeze(0), v_pool.unsqueeze(0), P)
+    DH, DD = max(width // 128, 1), 128                # the delta rule's heads
+    GH, GK, GV = max(width // 256, 1), 128, 256       # the gated linear attention beside it: as many state entries
+    for name, q_lens, ctx_lens in (("prefill 2048", [T], [T]), ("decode b8", [1] * B, [CTX] * B)):
+        n, prefill = sum(q_lens), q_lens[0] > 1
+        N = len(q_lens)
+        cu = i32([0] + list(torch.tensor(q_lens).cumsum(0)))
+        req = torch.repeat_interleave(torch.arange(N, dtype=torch.int32), torch.tensor(q_lens)).to(dev)
+        pos = i32(list(range(T)) if prefill else [CTX - 1] * B)
+        slots = i32([(r * (CTX // P)) * P + (i if prefill else CTX - 1) for r, x in enumerate(q_lens) for i in range(x)])
+        table = torch.stack([torch.arange(r * (CTX // P), r * (CTX // P) + CTX // P + 1, dtype=torch.int32) % n_pages for r in range(N)]).to(dev).contiguous()
+        state_slots = i32(list(range(N)))
+        step = dict(req_of_token=req, cu_q=cu, state_slots=state_slots)
+        # ---- the stream
+        stream, w, mu = torch.randn(n, width, device=dev), torch.ones(width, device=dev), torch.rand(width, device=dev)
+        x, x2 = rand(n, width), rand(n, width)
+        shift_state = torch.zeros(N, width, device=dev)
+        put(f"add_rms_norm {name}", None, lambda: ops.add_rms_norm(x, stream, w, 1e-6), bytes_=n * width * (2 + 4 + 4 + 2))
+        put(f"norm_add_norm {name}", f"add_rms_norm {name}", lambda: ops.norm_add_norm(stream, x, w, 1e-6, w, 1e-6), bytes_=n * width * (2 + 4 + 4 + 2))
+        put(f"shift_norm {name} (post-norm, add, norm, token shift)", f"norm_add_norm {name}",
+            lambda: ops.shift_norm(stream, w, 1e-6, mu, shift_state, bf, y=x, post_weight=w, post_eps=1e-6, **step),
+            bytes_=n * width * (2 + 4 + 4 + 2) + N * width * 8)
+        put(f"pair_norm_mean {name}", f"add_rms_norm {name}", lambda: ops.pair_norm_mean(x, x2, w, w, 1e-5), bytes_=n * width * 6)
+        put(f"scaled_sum {name}", f"pair_norm_mean {name}", lambda: ops.scaled_sum(x, x2, 0.7, 0.6), bytes_=n * width * 6)
+        # ---- between the products and attention
+        qkv = rand(n, cq + ck + cv, scale=0.5)
+        put(f"qk_norm_rope_store {name}", None,
+            lambda: ops.qk_norm_rope_store(qkv, ones, ones, cos_table, cos_table, pos, slots, k_pool, v_pool, H, KV, D, 1e-6, status), bytes_=n * (cq + ck + cv) * 4)
+        cos = torch.ones(n, D // 4, device=dev)
+        temp = torch.ones(H, device=dev)
+        put(f"head_prep {name} (q/k norm, half of each head rotated, temperature, cache write)", f"qk_norm_rope_store {name}",
+            lambda: ops.head_prep(qkv, q_col0=0, k_col0=cq, v_col0=cq + ck, num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=D, norm="weighted", q_weight=ones,
+                                  k_weight=ones, q_factor=temp, cos=cos, sin=cos, k_pool=k_pool, v_pool=v_pool, slots=slots, n_requests=N, status=status,
+                                  eps=1e-6, **step), bytes_=n * (cq + ck + cv) * 4)
+        bias = rand(cq + ck + cv, dtype=torch.float32)
+        put(f"diff_prep {name} (biases, two query rows per head, cache write)", f"qk_norm_rope_store {name}",
+            lambda: ops.diff_prep(qkv, num_heads=H, num_kv_heads=KV, dim=D // 2, value_dim=D, width=D, bias=bias, k_pool=k_pool, v_pool=v_pool, slots=slots,
+                                  status=status), bytes_=n * ((cq + ck + cv) * 2 + (2 * cq + ck + cv) * 2))
+        down = rand(n, QL + L + R)
+        qn, cn = torch.ones(QL, device=dev), torch.ones(L, device=dev)
+        put(f"cols_rms_norm {name} (the queries' latent, {QL} columns)", f"add_rms_norm {name}", lambda: ops.cols_rms_norm(down[:, :QL], qn, 1e-6), bytes_=n * QL * 4)
+        q_lat, q_abs = rand(n, H, D + R), torch.empty(n, H, L + R, dtype=bf, device=dev)
+        ang = torch.ones(n, R // 2, device=dev)
+        put(f"latent_prep {name} (latent row normed and stored, rotated parts)", f"qk_norm_rope_store {name}",
+            lambda: ops.latent_prep(latent_pool, down[:, QL:], L, R, cn, 1e-6, q_lat, H, D + R, D, q_abs, L + R, L, ang, ang, slots, status, halves=True),
+            bytes_=n * ((L + R) * 4 + H * R * 4))
+        # ---- the latent mixer's per-head maps
+        uk, uv = rand(H, D, L, scale=0.05), rand(H, L, D, scale=0.05)
+        o_lat, o_val = rand(n, H, L + R), torch.empty(n, H, D, dtype=bf, device=dev)
+        big = rand(H * D, L)
+        flat = rand(n, L)
+        wts = dict(flops=2 * n * H * D * L) if prefill else dict(bytes_=H * D * L * 2)
+        put(f"linear {name} (the same FLOPs as one product)", None, lambda: ops.linear(flat, big), **wts)
+        put(f"head_linear {name} (queries into the latent space)", f"linear {name} (the same FLOPs as one product)", lambda: ops.head_linear(q_abs, 0, q_lat, 0, uk), **wts)
+        put(f"head_linear {name} (latent output to values)", f"linear {name} (the same FLOPs as one product)", lambda: ops.head_linear(o_val, 0, o_lat, 0, uv), **wts)
+
+        # ---- attention
+        def tiles_for(spec):
+            r_ = [r for r, x_ in enumerate(q_lens) if spec[1] <= x_ <= spec[2] for _ in range(0, x_, spec[0])]
+            t_ = [t0 for r, x_ in enumerate(q_lens) if spec[1] <= x_ <= spec[2] for t0 in range(0, x_, spec[0])]
+            return i32(r_ + [0]), i32(t_ + [0]), len(r_)
+
+        positions = range(T) if prefill else [CTX - 1] * B
+        causal = sum(p + 1 for p in positions)
+        windowed = sum(min(p + 1, WINDOW) for p in positions)
+
+        def attention(label, like, heads_, kv_, k, v, *, tma, window=0, flops_per_key=None, bytes_per_key=None, **extras):
+            width_ = k.shape[-1]
+            specs = ops.attention_tile_specs(heads_, kv_, width_, bf, P if tma else None)
+            q = rand(n, heads_, width_)
+            args = dict(tiles={spec: tiles_for(spec) for spec in specs}, cu_q=cu, ctx_lens=i32(ctx_lens), block_table=table, page_size=P, scale=D ** -0.5,
+                        window=window, kv_len_bound=max(ctx_lens), status=status, kv_maps=maps if tma else None, **extras)
+            seen = windowed if window else causal
+            work = dict(flops=seen * (flops_per_key or 4 * heads_ * width_)) if prefill else dict(bytes_=seen * (bytes_per_key or kv_ * 2 * width_ * 2))
+            put(label, like, lambda: ops.paged_attention(q, k, v, **args), **work)
+
+        tma_kind, cp_kind = ("tcgen05, TMA", "cp.async mma") if prefill else ("TMA split-KV", "cp.async split-KV")
+        attention(f"paged_attention {name} ({tma_kind})", None, H, KV, k_pool, v_pool, tma=True)
+        attention(f"windowed attention {name} (last {WINDOW} keys; {tma_kind})", f"paged_attention {name} ({tma_kind})", H, KV, k_pool, v_pool, tma=True, window=WINDOW)
+        # the work of two maps of D / 2 and one value product each; the zero halves of the query rows are the kernel's own affair
+        attention(f"differential attention {name} (two maps per head, last {WINDOW} keys; {tma_kind})", f"windowed attention {name} (last {WINDOW} keys; {tma_kind})",
+                  2 * H, KV, k_pool, v_pool, tma=True, window=WINDOW, flops_per_key=2 * H * (D + 2 * D))
+        attention(f"paged_attention {name} ({cp_kind})", None, H, KV, k_pool, v_pool, tma=False)
+        sink = torch.zeros(H, device=dev)
+        attention(f"latent attention {name} with a sink (Radapel's; {cp_kind})", f"paged_attention {name} ({cp_kind})", H, 1, latent_pool, latent_pool, tma=False,
+                  bytes_per_key=(L + R) * 2, sink=sink)
+        attention(f"latent attention {name} (256-wide shared row; {cp_kind})", f"latent attention {name} with a sink (Radapel's; {cp_kind})", H, 1, latent_pool,
+                  latent_pool, tma=False, bytes_per_key=(L + R) * 2)
+        # ---- behind attention
+        o2, lam = rand(n, 2 * H, D), torch.full((1,), 0.4, device=dev)
+        o, gates, gates_pair = rand(n, H * D), rand(n, H), rand(n, 2 * H * D)
+        put(f"silu_mul {name} ({H * D} columns)", None, lambda: ops.silu_mul(gates_pair), bytes_=n * H * D * 6)
+        put(f"diff_combine {name} (difference of the maps, head norm)", f"silu_mul {name} ({H * D} columns)", lambda: ops.diff_combine(o2, H, D, lam, 1e-6, 0.6),
+            bytes_=n * H * D * 6)
+        put(f"sigmoid_gate {name} (a gate per head, in place)", f"silu_mul {name} ({H * D} columns)", lambda: ops.sigmoid_gate_(o, gates, 0, D, per_head=True),
+            bytes_=n * H * D * 4)
+        # ---- the recurrences
+        inner, keys = GH * GV, GH * GK
+        gproj = rand(n, 2 * keys + 2 * inner, scale=0.3)
+        z, zb = torch.randn(n, keys, device=dev), torch.full((keys,), 3.0, device=dev)
+        gstate = torch.zeros(N + 1, GH * GK * GV, device=dev)
+        put(f"gla_scan {name} ({GH} heads of {GK} x {GV})", None,
+            lambda: ops.gla_scan(gproj, 0, keys, 2 * keys, z, zb, heads=GH, key_dim=GK, value_dim=GV, tau=16.0, q_scale=GK ** -0.5, state=gstate, cu_q=cu,
+                                 state_slots=state_slots, n_requests=N),
+            bytes_=n * (2 * keys + inner) * 2 + n * keys * 4 + n * inner * 4 + N * GH * GK * GV * 8)
+        di = DH * DD
+        dproj, rates = rand(n, 4 * di, scale=0.3), torch.randn(n, di + 64, device=dev)
+        zw, vec = torch.randn(n, di, device=dev), torch.zeros(di, device=dev)
+        dstate = torch.zeros(N + 1, DH * DD * DD, device=dev)
+        put(f"delta_scan {name} ({DH} heads of {DD} x {DD})", f"gla_scan {name} ({GH} heads of {GK} x {GV})",
+            lambda: ops.delta_scan(dproj, 0, di, 2 * di, zw, vec, rates, vec, heads=DH, key_dim=DD, value_dim=DD, rate=0.6, len_eps=1e-6, state=dstate, cu_q=cu,
+                                   state_slots=state_slots, n_requests=N, single_tokens=not prefill),
+            bytes_=n * di * (3 * 2 + 2 * 4 + 4) + N * DH * DD * DD * 8)
+        put(f"tanh_cols {name} (64 columns)", f"silu_mul {name} ({H * D} columns)", lambda: ops.tanh_cols(rates, di, 64, bf), bytes_=n * 64 * 6)
+        y, wn = torch.randn(n, di, device=dev), torch.ones(di, device=dev)
+        put(f"head_norm_gate {name} ({GH} heads of {GV})", None, lambda: ops.head_norm_gate(y, dproj, 3 * di, wn, GH, 1e-6), bytes_=n * di * 8)
+        put(f"head_norm_gate {name} ({DH} heads of {DD})", f"head_norm_gate {name} ({GH} heads of {GV})", lambda: ops.head_norm_gate(y, dproj, 3 * di, wn, DH, 1e-6),
+            bytes_=n * di * 8)
+        # ---- the router
+        E, ID, top = 16, 4, 4
+        zr, corr, kept = torch.randn(n, E + ID, device=dev), torch.zeros(E + ID, device=dev), torch.empty(n, device=dev)
+        put(f"route {name} (softmax of {E + ID})", None, lambda: ops.route(zr, top=top, groups=1, keep=1, scale=1.0, score="softmax", renormalize=False),
+            bytes_=n * (2 * (E + ID) + 2 * top) * 4)
+        put(f"route {name} (softmax of {E + ID}, correction, {ID} identity experts)", f"route {name} (softmax of {E + ID})",
+            lambda: ops.route(zr, top=top, groups=1, keep=1, scale=1.0, score="softmax", renormalize=False, correction=corr, kept=kept, identity=ID),
+            bytes_=n * (2 * (E + ID) + 2 * top) * 4)
+    # ---- the feed-forwards as a whole
+    from oxr_inference_b200.parts.base import FEED_FORWARDS, Runtime
+
+    rt = Runtime(device=torch.device(dev), dtype=bf, max_positions=1, status=status)
+    E, ID, top, ffe = 16, 4, 4, ff // 8
+
+    def built(kind, **params):
+        part = FEED_FORWARDS.build(kind, rt, hidden_size=width, **params)
+        for pname, info in part.parameters().items():
+            part.assign(pname, rand(*info.shape, scale=0.02))
+        part.finish_loading()
+        return part
+
+    swiglu, gelu = built("swiglu", intermediate_size=ff), built("gelu_glu", intermediate_size=ff)
+    common = dict(intermediate_size=ffe, experts=E, top=top, activation="silu_glu", score="softmax", renormalize=False)
+    plain_moe, moe = built("routed_experts", **common), built("routed_experts", choice_correction=True, identity=ID, **common)
+    for n in (T, B):
+        h = rand(n, width)
+        work = dict(flops=2 * n * width * 3 * ff) if n >= 256 else dict(bytes_=3 * ff * width * 2)
+        put(f"SiLU-gated feed-forward {n} rows ({ff})", None, lambda: swiglu.forward(h), **work)
+        put(f"GELU-gated feed-forward {n} rows ({ff})", f"SiLU-gated feed-forward {n} rows ({ff})", lambda: gelu.forward(h), **work)
+        for label, part, like, share in ((f"routed experts {n} rows ({top} of {E} of {ffe})", plain_moe, f"SiLU-gated feed-forward {n} rows ({ff})", 1.0),
+                                         (f"routed experts {n} rows ({top} of {E} of {ffe} and {ID} identity)", moe, f"routed experts {n} rows ({top} of {E} of {ffe})",
+                                          E / (E + ID))):
+            touched = E * (1 - (1 - share * top / E) ** n)
+            put(label, like, lambda: part.forward(h), **(dict(flops=2 * n * width * 3 * ffe * top * share) if n >= 256 else dict(bytes_=3 * width * 2 * touched * ffe)))
+    ops.check_status(status)
+    return rows
+
+
+def verorax_workload(args) -> int:
+    """The Verorax design beside Nidudra (the closest design: pairs of mixers, a recurrence, routed experts) and Qwen3 at equal sizes: whole-model
+    prefill and decode throughput at two sizes, and every kernel of its parts against its roofline beside the like kernel."""
+    import torch
+
+    sizes = [("2048 wide, 8 layers", dict(width=2048, ff=8192, heads=16, kv_heads=4, head_dim=128, layers=8, vocab=32768)),
+             ("4096 wide, 8 layers (Qwen3-8B layer sizes)", dict(width=4096, ff=12288, heads=32, kv_heads=8, head_dim=128, layers=8, vocab=32768))]
+    K, W = args.steps, max(args.warmup, 3)
+    sampler = ClockSampler()
+    sampler.start()
+    out = {"workload": "verorax", "dtype": "bf16", "data": "synthetic uniform token ids, random weights N(0, 0.02)", "steps": K, "warmup": W,
+           "batch": 8, "context": args.context, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks()[2], "sizes": []}
+    for name, s in sizes:
+        qwen = {"architectures": ["Qwen3ForCausalLM"], "model_type": "qwen3", "hidden_size": s["width"], "intermediate_size": s["ff"],
+                "num_hidden_layers": s["layers"], "num_attention_heads": s["heads"], "num_key_value_heads": s["kv_heads"], "head_dim": s["head_dim"],
+                "rms_norm_eps": 1e-6, "rope_theta": 1000000.0, "vocab_size": s["vocab"], "tie_word_embeddings": False,
+                "max_position_embeddings": 8192}
+        row = {"size": name}
+        for design, cfg in (("qwen3", qwen), ("nidudra", nidudra_config(**s)), ("verorax", verorax_config(**s))):
+            row[design] = design_throughput(cfg, s["vocab"], K, W, 8, args.context, PREFILL_TOKENS)
+            torch.cuda.empty_cache()
+        out["sizes"].append(row)
+    last = sizes[-1][1]
+    out["kernels"] = verorax_kernels(last["width"], last["heads"], last["kv_heads"], last["head_dim"], last["ff"])
+    out["clocks"] = sampler.stop()
+    print(json.dumps(out))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1037,9 +1280,9 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64 and the further points (quick runs)")
     ap.add_argument("--skip-serving", action="store_true", help="leave the two serving workloads out of `points`")
     ap.add_argument("--context", type=int, default=CONTEXT, help="tokens each request holds when the decode steps are timed")
-    ap.add_argument("--workload", default="decode", choices=("decode", "continuous", "chunked", "radapel", "bifusun", "vazepel", "nidudra"),
+    ap.add_argument("--workload", default="decode", choices=("decode", "continuous", "chunked", "radapel", "bifusun", "vazepel", "nidudra", "verorax"),
                     help="decode: the headline line (default); continuous / chunked: the two serving workloads, one line each; "
-                         "radapel / bifusun / vazepel / nidudra: that design beside Qwen3 at equal sizes, whole models and kernel by kernel")
+                         "radapel / bifusun / vazepel / nidudra / verorax: that design beside Qwen3 (verorax: and Nidudra) at equal sizes, whole models and kernel by kernel")
     args = ap.parse_args()
     if args.gpus != 1:
         print(f"this engine runs on one GPU; --gpus {args.gpus} is not supported")
@@ -1054,6 +1297,8 @@ def main() -> int:
         return vazepel_workload(args)
     if args.workload == "nidudra":
         return nidudra_workload(args)
+    if args.workload == "verorax":
+        return verorax_workload(args)
     if args.workload != "decode":
         return serving_workload(args.workload)
     K, W = args.steps, max(args.warmup, 3)

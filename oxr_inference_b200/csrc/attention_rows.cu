@@ -211,11 +211,141 @@ __global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, 
         }
 }
 
+// The same for bf16 and half-split pairs, everything whole 16-byte words (rank, rot, half, strides and offsets multiples of 8; rot == 2 half). Warp 0
+// writes the cache row; every thread then takes one pair of words (w and w + half / 8 of a rotated part) and walks over the heads with its
+// angles in registers.
+__device__ __forceinline__ void lp_unpack(const uint4& v, float (&out)[8]) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = __bfloat1622float2(h[i]);
+        out[2 * i] = f.x; out[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ uint4 lp_pack(const float (&v)[8]) {
+    uint4 out;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    return out;
+}
+__device__ __forceinline__ void lp_load8(const float* p, float (&out)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    out[0] = a.x; out[1] = a.y; out[2] = a.z; out[3] = a.w; out[4] = b.x; out[5] = b.y; out[6] = b.z; out[7] = b.w;
+}
+// (u, v) -> (u cos - v sin, v cos + u sin) for the words at p and p + half
+__device__ __forceinline__ void lp_turn(__nv_bfloat16* dst, const __nv_bfloat16* src, int half, const float (&c)[8], const float (&s)[8]) {
+    float u[8], v[8], a[8], b[8];
+    lp_unpack(*reinterpret_cast<const uint4*>(src), u);
+    lp_unpack(*reinterpret_cast<const uint4*>(src + half), v);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        a[i] = u[i] * c[i] - v[i] * s[i];
+        b[i] = v[i] * c[i] + u[i] * s[i];
+    }
+    *reinterpret_cast<uint4*>(dst) = lp_pack(a);
+    *reinterpret_cast<uint4*>(dst + half) = lp_pack(b);
+}
+
+__global__ void __launch_bounds__(128) latent_prep_words_kernel(__nv_bfloat16* __restrict__ pool, long long slot_stride, long long pool_slots,
+                                                                const __nv_bfloat16* __restrict__ down, int down_stride, int rank,
+                                                                const float* __restrict__ weight, float eps, const __nv_bfloat16* q, int heads,
+                                                                int q_head_dim, int q_rot0, __nv_bfloat16* q_out, int qo_head_dim, int qo_rot0,
+                                                                const float* __restrict__ cos_t, const float* __restrict__ sin_t, int half,
+                                                                const int* __restrict__ slots, int* status) {
+    const int t = blockIdx.x, lane = threadIdx.x & 31, slot = slots[t], per = half / 8;     // words of half a rotated part
+    const __nv_bfloat16* row = down + (size_t)t * down_stride;
+    const float* ct = cos_t + (size_t)t * half;
+    const float* st = sin_t + (size_t)t * half;
+    if (threadIdx.x < 32) {
+        if (slot >= pool_slots) {
+            if (lane == 0) oxr_report(status, OXR_BAD_SLOT, t);
+        } else if (slot >= 0) {
+            float ss = 0.f, x[8];
+            for (int i = lane; i < rank / 8; i += 32) {
+                lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), x);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) ss = fmaf(x[k], x[k], ss);
+            }
+            const float inv = 1.f / sqrtf(warp_sum(ss) / (float)rank + eps);
+            __nv_bfloat16* dst = pool + (long long)slot * slot_stride;
+            for (int i = lane; i < rank / 8; i += 32) {
+                float w[8];
+                lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), x);
+                lp_load8(weight + 8 * i, w);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) x[k] = x[k] * inv * w[k];
+                *reinterpret_cast<uint4*>(dst + 8 * i) = lp_pack(x);
+            }
+            for (int i = lane; i < per; i += 32) {
+                float c[8], s[8];
+                lp_load8(ct + 8 * i, c);
+                lp_load8(st + 8 * i, s);
+                lp_turn(dst + rank + 8 * i, row + rank + 8 * i, half, c, s);
+            }
+        }
+    }
+    const int w = threadIdx.x % per, stride = blockDim.x / per;      // one word per thread; stride threads with the same word share the heads
+    if ((int)threadIdx.x < stride * per) {
+        float c[8], s[8];
+        lp_load8(ct + 8 * w, c);
+        lp_load8(st + 8 * w, s);
+        for (int h = threadIdx.x / per; h < heads; h += stride)
+            lp_turn(q_out + ((size_t)t * heads + h) * qo_head_dim + qo_rot0 + 8 * w, q + ((size_t)t * heads + h) * q_head_dim + q_rot0 + 8 * w, half, c, s);
+    }
+}
+
+__global__ void __launch_bounds__(128) cols_rms_norm_words_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, int stride, int width,
+                                                                  const float* __restrict__ weight, float eps) {
+    __shared__ float red[32];
+    const __nv_bfloat16* row = x + (size_t)blockIdx.x * stride;
+    constexpr int KEEP = 2;
+    float v[KEEP][8], ss = 0.f;
+    const int nw = width / 8;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int i = threadIdx.x + k * 128;
+        if (i < nw) {
+            lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), v[k]);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(v[k][e], v[k][e], ss);
+        }
+    }
+    for (int i = threadIdx.x + KEEP * 128; i < nw; i += 128) {
+        float y[8];
+        lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)width + eps);
+    for (int i = threadIdx.x, k = 0; i < nw; i += 128, ++k) {
+        float y[8], w[8];
+        if (k < KEEP) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y[e] = k == 0 ? v[0][e] : v[1][e];
+        } else {
+            lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), y);
+        }
+        lp_load8(weight + 8 * i, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) y[e] = y[e] * inv * w[e];
+        *reinterpret_cast<uint4*>(out + (size_t)blockIdx.x * width + 8 * i) = lp_pack(y);
+    }
+}
+
 OXR_API int oxr_latent_prep(void* pool, long long slot_stride, long long pool_slots, const void* down, int down_stride, int rank, int rot, const float* weight, float eps,
                             const void* q, int heads, int q_head_dim, int q_rot0, void* q_out, int qo_head_dim, int qo_rot0, const float* cos_t,
                             const float* sin_t, int half, int halves, const int* slots, int n_tokens, int dtype, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank <= 0 || down_stride < rank + rot || rot < 0 || 2 * half > rot || q_rot0 + rot > q_head_dim || qo_rot0 + rot > qo_head_dim) return OXR_BAD_ARGUMENT;
+    if (dtype == 1 && halves && half > 0 && half % 8 == 0 && half <= 1024 && rot == 2 * half && rank % 8 == 0 && slot_stride % 8 == 0 && down_stride % 8 == 0 &&
+        q_head_dim % 8 == 0 && q_rot0 % 8 == 0 && qo_head_dim % 8 == 0 && qo_rot0 % 8 == 0 && (uintptr_t)pool % 16 == 0 && (uintptr_t)down % 16 == 0 &&
+        (uintptr_t)q % 16 == 0 && (uintptr_t)q_out % 16 == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)cos_t % 16 == 0 && (uintptr_t)sin_t % 16 == 0) {
+        latent_prep_words_kernel<<<n_tokens, 128, 0, stream>>>((__nv_bfloat16*)pool, slot_stride, pool_slots, (const __nv_bfloat16*)down, down_stride, rank, weight,
+                                                              eps, (const __nv_bfloat16*)q, heads, q_head_dim, q_rot0, (__nv_bfloat16*)q_out, qo_head_dim, qo_rot0,
+                                                              cos_t, sin_t, half, slots, status);
+        return oxr_launch_status();
+    }
     if (dtype == 0)
         latent_prep_kernel<float><<<n_tokens, 128, 0, stream>>>((float*)pool, slot_stride, pool_slots, (const float*)down, down_stride, rank, rot, weight, eps, (const float*)q, heads,
                                                                q_head_dim, q_rot0, (float*)q_out, qo_head_dim, qo_rot0, cos_t, sin_t, half, halves, slots, status);
@@ -243,6 +373,10 @@ __global__ void cols_rms_norm_kernel(T* __restrict__ out, const T* __restrict__ 
 OXR_API int oxr_cols_rms_norm(void* out, const void* x, int n, int stride, int width, const float* weight, float eps, int dtype, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (width <= 0 || stride < width) return OXR_BAD_ARGUMENT;
+    if (dtype == 1 && width % 8 == 0 && stride % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)weight % 16 == 0) {
+        cols_rms_norm_words_kernel<<<n, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, stride, width, weight, eps);
+        return oxr_launch_status();
+    }
     const int threads = width >= 1024 ? 256 : 128;
     if (dtype == 0) cols_rms_norm_kernel<float><<<n, threads, 0, stream>>>((float*)out, (const float*)x, stride, width, weight, eps);
     else cols_rms_norm_kernel<__nv_bfloat16><<<n, threads, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)x, stride, width, weight, eps);
@@ -278,6 +412,54 @@ __global__ void __launch_bounds__(128) head_linear_kernel(T* __restrict__ out, i
     }
 }
 
+// The same for the few tokens of a decode step: a block takes TM tokens, one head and 64 output columns, its four warps a quarter of the inputs
+// each (a lane two neighbouring columns, eight rows of w asked for ahead); the quarters' sums are added in their order. n_out even.
+__device__ __forceinline__ float2 hl_load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 hl_load2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+
+template <typename T, int TM>
+__global__ void __launch_bounds__(128) head_linear_few_kernel(T* __restrict__ out, int out_head_stride, int out0, const T* __restrict__ x, int x_head_stride,
+                                                              int x0, const T* __restrict__ w, int n_in, int n_out, int heads, int n_tokens) {
+    extern __shared__ float xs[];   // [TM, n_in], then [4][TM][64]
+    float* part = xs + TM * n_in;
+    const int h = blockIdx.y, t0 = blockIdx.x * TM, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = blockIdx.z * 64 + 2 * lane;
+    for (int i = threadIdx.x; i < TM * n_in; i += 128) {
+        const int m = i / n_in, k = i - m * n_in;
+        xs[i] = (t0 + m < n_tokens) ? Num<T>::to_f32(x[((size_t)(t0 + m) * heads + h) * x_head_stride + x0 + k]) : 0.f;
+    }
+    __syncthreads();
+    const int per = (n_in + 3) / 4, k0 = min(n_in, warp * per), k1 = min(n_in, k0 + per);
+    const T* wh = w + (size_t)h * n_in * n_out + (c < n_out ? c : 0);
+    float acc[TM][2];
+#pragma unroll
+    for (int m = 0; m < TM; ++m) acc[m][0] = acc[m][1] = 0.f;
+    for (int k = k0; k < k1; k += 8) {
+        float2 wv[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) wv[i] = k + i < k1 ? hl_load2(wh + (size_t)(k + i) * n_out) : make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            if (k + i >= k1) break;
+#pragma unroll
+            for (int m = 0; m < TM; ++m) {
+                const float xv = xs[m * n_in + k + i];
+                acc[m][0] = fmaf(xv, wv[i].x, acc[m][0]);
+                acc[m][1] = fmaf(xv, wv[i].y, acc[m][1]);
+            }
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < TM; ++m) *reinterpret_cast<float2*>(part + (warp * TM + m) * 64 + 2 * lane) = make_float2(acc[m][0], acc[m][1]);
+    __syncthreads();
+    for (int i = threadIdx.x; i < TM * 64; i += 128) {
+        const int m = i / 64, o = blockIdx.z * 64 + i % 64;
+        if (t0 + m < n_tokens && o < n_out) {
+            const float v = ((part[i] + part[TM * 64 + i]) + part[2 * TM * 64 + i]) + part[3 * TM * 64 + i];
+            out[((size_t)(t0 + m) * heads + h) * out_head_stride + out0 + o] = Num<T>::from_f32(v);
+        }
+    }
+}
+
 // The same on the tensor cores (bf16, fp32 sums in k order per 16-wide step): a block takes 64 tokens of one head, a warp 16 of them;
 // x rows and the head's matrix, 64 output columns at a time, stand in shared memory. n_in a multiple of 16, n_out of 16.
 __device__ __forceinline__ void hl_ldsm_x4(uint32_t (&r)[4], const __nv_bfloat16* p) {
@@ -297,23 +479,40 @@ constexpr int HL_BM = 64, HL_BN = 64;
 
 __global__ void __launch_bounds__(128) head_linear_mma_kernel(__nv_bfloat16* __restrict__ out, int out_head_stride, int out0,
                                                               const __nv_bfloat16* __restrict__ x, int x_head_stride, int x0,
-                                                              const __nv_bfloat16* __restrict__ w, int n_in, int n_out, int heads, int n_tokens) {
+                                                              const __nv_bfloat16* __restrict__ w, int n_in, int n_out, int heads, int n_tokens, int words) {
     extern __shared__ __align__(16) unsigned char hl_smem[];
     const int lda = n_in + 8, ldb = HL_BN + 8;
     __nv_bfloat16* As = reinterpret_cast<__nv_bfloat16*>(hl_smem);   // [64][n_in + 8]
     __nv_bfloat16* Bs = As + HL_BM * lda;                            // [n_in][64 + 8]
     const int h = blockIdx.y, t0 = blockIdx.x * HL_BM, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int i = threadIdx.x; i < HL_BM * n_in; i += 128) {
-        const int m = i / n_in, k = i % n_in;
-        As[m * lda + k] = (t0 + m < n_tokens) ? x[((size_t)(t0 + m) * heads + h) * x_head_stride + x0 + k] : __float2bfloat16_rn(0.f);
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    if (words) {      // rows of x and of w are whole 16-byte words
+        const int nk = n_in / 8;
+        for (int i = threadIdx.x; i < HL_BM * nk; i += 128) {
+            const int m = i / nk, k = (i - m * nk) * 8;
+            *reinterpret_cast<uint4*>(As + m * lda + k) =
+                (t0 + m < n_tokens) ? *reinterpret_cast<const uint4*>(x + ((size_t)(t0 + m) * heads + h) * x_head_stride + x0 + k) : zero;
+        }
+    } else {
+        for (int i = threadIdx.x; i < HL_BM * n_in; i += 128) {
+            const int m = i / n_in, k = i % n_in;
+            As[m * lda + k] = (t0 + m < n_tokens) ? x[((size_t)(t0 + m) * heads + h) * x_head_stride + x0 + k] : __float2bfloat16_rn(0.f);
+        }
     }
     const __nv_bfloat16* wh = w + (size_t)h * n_in * n_out;
-    for (int c0 = 0; c0 < n_out; c0 += HL_BN) {
+    for (int c0 = blockIdx.z * HL_BN; c0 < n_out; c0 += gridDim.z * HL_BN) {
         const int cols = min(HL_BN, n_out - c0);
         __syncthreads();   // As is in; the previous chunk's Bs is no longer read
-        for (int i = threadIdx.x; i < n_in * HL_BN; i += 128) {
-            const int k = i / HL_BN, c = i % HL_BN;
-            Bs[k * ldb + c] = c < cols ? wh[(size_t)k * n_out + c0 + c] : __float2bfloat16_rn(0.f);
+        if (words) {
+            for (int i = threadIdx.x; i < n_in * (HL_BN / 8); i += 128) {
+                const int k = i / (HL_BN / 8), c = (i % (HL_BN / 8)) * 8;
+                *reinterpret_cast<uint4*>(Bs + k * ldb + c) = c < cols ? *reinterpret_cast<const uint4*>(wh + (size_t)k * n_out + c0 + c) : zero;
+            }
+        } else {
+            for (int i = threadIdx.x; i < n_in * HL_BN; i += 128) {
+                const int k = i / HL_BN, c = i % HL_BN;
+                Bs[k * ldb + c] = c < cols ? wh[(size_t)k * n_out + c0 + c] : __float2bfloat16_rn(0.f);
+            }
         }
         __syncthreads();
         float acc[HL_BN / 8][4];
@@ -338,8 +537,12 @@ __global__ void __launch_bounds__(128) head_linear_mma_kernel(__nv_bfloat16* __r
 #pragma unroll
             for (int i = 0; i < HL_BN / 8; ++i)
                 if (i * 8 + 2 * (lane & 3) < cols) {
-                    dst[i * 8] = __float2bfloat16_rn(acc[i][2 * r]);
-                    dst[i * 8 + 1] = __float2bfloat16_rn(acc[i][2 * r + 1]);
+                    if (words) {
+                        *reinterpret_cast<__nv_bfloat162*>(dst + i * 8) = __floats2bfloat162_rn(acc[i][2 * r], acc[i][2 * r + 1]);
+                    } else {
+                        dst[i * 8] = __float2bfloat16_rn(acc[i][2 * r]);
+                        dst[i * 8 + 1] = __float2bfloat16_rn(acc[i][2 * r + 1]);
+                    }
                 }
         }
     }
@@ -358,8 +561,22 @@ OXR_API int oxr_head_linear(void* out, int out_head_stride, int out0, const void
             configured = mma_smem;
         }
         dim3 grid((n_tokens + HL_BM - 1) / HL_BM, heads);
+        const int words = x_head_stride % 8 == 0 && x0 % 8 == 0 && out_head_stride % 2 == 0 && out0 % 2 == 0 && (uintptr_t)x % 16 == 0 &&
+                          (uintptr_t)w % 16 == 0 && (uintptr_t)out % 4 == 0;
         head_linear_mma_kernel<<<grid, 128, mma_smem, stream>>>((__nv_bfloat16*)out, out_head_stride, out0, (const __nv_bfloat16*)x, x_head_stride, x0,
-                                                               (const __nv_bfloat16*)w, n_in, n_out, heads, n_tokens);
+                                                               (const __nv_bfloat16*)w, n_in, n_out, heads, n_tokens, words);
+        return oxr_launch_status();
+    }
+    constexpr int FEW = 8;
+    const size_t few_smem = (size_t)(FEW * n_in + 4 * FEW * 64) * sizeof(float);
+    if (n_tokens <= 16 && n_out % 2 == 0 && few_smem <= 48 * 1024 && (uintptr_t)w % 8 == 0) {
+        dim3 grid((n_tokens + FEW - 1) / FEW, heads, (n_out + 63) / 64);
+        if (dtype == 0)
+            head_linear_few_kernel<float, FEW><<<grid, 128, few_smem, stream>>>((float*)out, out_head_stride, out0, (const float*)x, x_head_stride, x0, (const float*)w,
+                                                                                n_in, n_out, heads, n_tokens);
+        else
+            head_linear_few_kernel<__nv_bfloat16, FEW><<<grid, 128, few_smem, stream>>>((__nv_bfloat16*)out, out_head_stride, out0, (const __nv_bfloat16*)x,
+                                                                                        x_head_stride, x0, (const __nv_bfloat16*)w, n_in, n_out, heads, n_tokens);
         return oxr_launch_status();
     }
     constexpr int TM = 8;

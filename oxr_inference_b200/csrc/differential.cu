@@ -116,15 +116,15 @@ OXR_API int oxr_diff_prep(void* q_out, void* k_pool, void* v_pool, const void* p
     return oxr_launch_status();
 }
 
-// one warp per (token, head); the head's entries stay in registers when they fit (DV <= 32 * VEC * 4 words a lane), else they are computed twice
-template <typename T, int VEC>
+// G lanes per (token, head), G a power of two: the head's entries stay in registers when they fit (KEEP words a lane), else they are read twice
+template <typename T, int VEC, int G>
 __global__ void __launch_bounds__(128) diff_combine_kernel(T* __restrict__ out, const T* __restrict__ o, int o_head, int H, int DV, const float* __restrict__ lambda,
                                                            float eps, float factor, int n_tokens) {
-    const int lane = threadIdx.x & 31;
-    const long long at = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (at >= (long long)n_tokens * H) return;
+    const int l = threadIdx.x % G;
+    const long long at = (long long)blockIdx.x * (128 / G) + threadIdx.x / G;
+    const bool live = at < (long long)n_tokens * H;      // the others walk along: the sums are for whole warps
     const float lam = *lambda;
-    const T* o1 = o + at * 2 * o_head;
+    const T* o1 = o + (live ? at : 0) * 2 * o_head;
     const T* o2 = o1 + o_head;
     constexpr int KEEP = 4;
     DiffWord<T, VEC> kept[KEEP];
@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(128) diff_combine_kernel(T* __restrict__ out, 
     float sq = 0.f;
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
-        const int w = lane + 32 * k;
+        const int w = l + G * k;
         if (w < nw) {
             DiffWord<T, VEC> b;
             kept[k].load(o1 + w * VEC);
@@ -144,7 +144,7 @@ __global__ void __launch_bounds__(128) diff_combine_kernel(T* __restrict__ out, 
             }
         }
     }
-    for (int w = lane + 32 * KEEP; w < nw; w += 32) {
+    for (int w = l + G * KEEP; w < nw; w += G) {
         DiffWord<T, VEC> a, b;
         a.load(o1 + w * VEC);
         b.load(o2 + w * VEC);
@@ -154,18 +154,21 @@ __global__ void __launch_bounds__(128) diff_combine_kernel(T* __restrict__ out, 
             sq = fmaf(v, v, sq);
         }
     }
-    const float inv = factor / sqrtf(warp_sum(sq) / (float)DV + eps);
+#pragma unroll
+    for (int s = G >> 1; s > 0; s >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, s);
+    if (!live) return;
+    const float inv = factor / sqrtf(sq / (float)DV + eps);
     T* dst = out + at * DV;
 #pragma unroll
     for (int k = 0; k < KEEP; ++k) {
-        const int w = lane + 32 * k;
+        const int w = l + G * k;
         if (w < nw) {
 #pragma unroll
             for (int i = 0; i < VEC; ++i) kept[k].v[i] *= inv;
             kept[k].store(dst + w * VEC);
         }
     }
-    for (int w = lane + 32 * KEEP; w < nw; w += 32) {
+    for (int w = l + G * KEEP; w < nw; w += G) {
         DiffWord<T, VEC> a, b;
         a.load(o1 + w * VEC);
         b.load(o2 + w * VEC);
@@ -179,12 +182,19 @@ OXR_API int oxr_diff_combine(void* out, const void* o, int n_tokens, int o_head,
                              cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (H <= 0 || DV <= 0 || o_head < DV) return OXR_BAD_ARGUMENT;
-    const unsigned blocks = (unsigned)(((long long)n_tokens * H + 3) / 4);
-    if (dtype == 1 && DV % 8 == 0 && o_head % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)o % 16 == 0)
-        diff_combine_kernel<__nv_bfloat16, 8><<<blocks, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)o, o_head, H, DV, lambda, eps, factor, n_tokens);
-    else if (dtype == 0)
-        diff_combine_kernel<float, 1><<<blocks, 128, 0, stream>>>((float*)out, (const float*)o, o_head, H, DV, lambda, eps, factor, n_tokens);
-    else
-        diff_combine_kernel<__nv_bfloat16, 1><<<blocks, 128, 0, stream>>>((__nv_bfloat16*)out, (const __nv_bfloat16*)o, o_head, H, DV, lambda, eps, factor, n_tokens);
+    const long long total = (long long)n_tokens * H;
+#define OXR_COMBINE(T, VEC, G) \
+    diff_combine_kernel<T, VEC, G><<<(unsigned)((total + 128 / G - 1) / (128 / G)), 128, 0, stream>>>((T*)out, (const T*)o, o_head, H, DV, lambda, eps, factor, n_tokens)
+    if (dtype == 1 && DV % 8 == 0 && o_head % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)o % 16 == 0) {
+        // two words a lane where a head has that many
+        if (DV <= 128) OXR_COMBINE(__nv_bfloat16, 8, 8);
+        else if (DV <= 256) OXR_COMBINE(__nv_bfloat16, 8, 16);
+        else OXR_COMBINE(__nv_bfloat16, 8, 32);
+    } else if (dtype == 0) {
+        OXR_COMBINE(float, 1, 32);
+    } else {
+        OXR_COMBINE(__nv_bfloat16, 1, 32);
+    }
+#undef OXR_COMBINE
     return oxr_launch_status();
 }

@@ -2057,7 +2057,7 @@ def tanh_cols(z: torch.Tensor, col0: int, width: int, out_dtype: torch.dtype) ->
 
 def delta_scan(proj: torch.Tensor, r_col0: int, k_col0: int, v_col0: int, zw: torch.Tensor, w_bias: torch.Tensor, za: torch.Tensor, a_bias: torch.Tensor, *,
                heads: int, key_dim: int, value_dim: int, rate: float, len_eps: float, state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
-               n_requests: int, columns_per_thread: int = 0) -> torch.Tensor:
+               n_requests: int, single_tokens: bool = False) -> torch.Tensor:
     """The delta rule with a decay per key channel over a packed step: per head, with ``u = k / sqrt(sum k^2 + len_eps)``, ``w = exp(-rate *
     sigmoid(zw + w_bias))`` and ``a = sigmoid(za + a_bias)``,
 
@@ -2065,8 +2065,8 @@ def delta_scan(proj: torch.Tensor, r_col0: int, k_col0: int, v_col0: int, zw: to
 
     ``proj`` holds r, k and v head by head from the given columns; ``zw`` and ``za`` (fp32 ``[tokens, >= heads * key_dim]``, the first columns) are the
     logits of decay and removal rate; ``state`` (fp32, first axis the slot: S transposed, ``[heads, value_dim, key_dim]``) is read and left at the
-    state after each request's last token. Returns fp32 ``o [tokens, heads * value_dim]``. ``columns_per_thread`` (1 or 2) forces the kernel's
-    split; 0 chooses by the step's shape."""
+    state after each request's last token. ``single_tokens``: every request brings exactly one token (a decode step has a kernel of its own).
+    Returns fp32 ``o [tokens, heads * value_dim]``."""
     _need(proj, "proj")
     _need(zw, "zw", torch.float32)
     _need(za, "za", torch.float32)
@@ -2084,7 +2084,7 @@ def delta_scan(proj: torch.Tensor, r_col0: int, k_col0: int, v_col0: int, zw: to
     _done(_lib().oxr_delta_scan(y.data_ptr(), proj.data_ptr(), int(n_requests), proj.shape[1], int(r_col0), int(k_col0), int(v_col0), zw.data_ptr(),
                                 zw.shape[1], w_bias.data_ptr(), za.data_ptr(), za.shape[1], a_bias.data_ptr(), float(rate), float(len_eps), int(heads),
                                 int(key_dim), int(value_dim), state.data_ptr(), state.stride(0), cu_q.data_ptr(), state_slots.data_ptr(),
-                                _dtype_code(proj), int(columns_per_thread or 1), _stream()), "delta_scan")
+                                int(bool(single_tokens)), _dtype_code(proj), _stream()), "delta_scan")
     return y
 
 

@@ -67,5 +67,5 @@ class DeltaRule(Mixer):
         z = self.decay(ops.tanh_cols(rates, self.inner, self.rank, h.dtype), torch.float32)
         o = ops.delta_scan(proj, 0, self.inner, 2 * self.inner, z, v["w0"], rates, v["a.b"], heads=self.H, key_dim=self.D, value_dim=self.D,
                            rate=self.rate, len_eps=self.length_eps, state=cache.state, cu_q=ctx.cu_q, state_slots=ctx.state_slots,
-                           n_requests=ctx.n_requests)
+                           n_requests=ctx.n_requests, single_tokens=ctx.single_tokens)
         return self.out(ops.head_norm_gate(o, proj, 3 * self.inner, v["norm"], self.H, self.eps))
