@@ -272,33 +272,33 @@ __global__ void __launch_bounds__(128) head_prep_bf16x8_kernel(__nv_bfloat16* __
     }
 }
 
-// The same without a filter, for steps of many tokens: a group of DK / 8 lanes takes HPG heads of one token one after the other, so that the
+// The same without a filter, for steps of many tokens and heads of 64 or 128 entries: a group of LPH = DK / 8 lanes takes HPG heads of one token one after the other, so that the
 // token's angles, which every head turns by, are fetched once for all of them and the heads' loads are in flight together.
-template <int HPG>
-__global__ void __launch_bounds__(128) head_prep_heads_kernel(__nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_pool,
-                                                              __nv_bfloat16* __restrict__ v_pool, const __nv_bfloat16* __restrict__ proj, const PrepArgs a,
-                                                              int lph, int hpw) {
+template <int LPH, int HPG>
+__global__ void __launch_bounds__(128, HPG == 2 ? 8 : 5) head_prep_heads_kernel(__nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_pool,
+                                                              __nv_bfloat16* __restrict__ v_pool, const __nv_bfloat16* __restrict__ proj, const PrepArgs a) {
     using bf16 = __nv_bfloat16;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, groups = (blockDim.x >> 5) * hpw;
+    constexpr int HPW = 32 / LPH, GROUPS = 4 * HPW, DK = 8 * LPH;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x;
-    const int sub = lane / lph, l = lane - sub * lph, g0 = sub * lph;
+    const int sub = lane / LPH, l = lane % LPH;
     const int n_k = a.has_k ? a.KV : 0, n_v = a.v_mode == 1 ? a.KV : 0;
     const int slot = a.slots[t];
     const bf16* row = proj + (size_t)t * a.stride;
-    const int head0 = (blockIdx.y * groups + warp * hpw + sub), step = groups * gridDim.y;   // this group's heads: head0 + i step
+    const int head0 = blockIdx.y * GROUPS + warp * HPW + sub, step = GROUPS * gridDim.y;   // this group's heads: head0 + i step
     uint4 raw[HPG];
 #pragma unroll
     for (int i = 0; i < HPG; ++i) {
         const int head = head0 + i * step;
-        const bool live = sub < hpw && head < a.H + n_k + n_v && (head < a.H + n_k || 8 * l < a.DV);
-        const int col = head < a.H ? a.q_col0 + head * a.DK : (head < a.H + n_k ? a.k_col0 + (head - a.H) * a.DK : a.v_col0 + (head - a.H - n_k) * a.DV);
+        const bool live = head < a.H + n_k + n_v && (head < a.H + n_k || 8 * l < a.DV);
+        const int col = head < a.H ? a.q_col0 + head * DK : (head < a.H + n_k ? a.k_col0 + (head - a.H) * DK : a.v_col0 + (head - a.H - n_k) * a.DV);
         raw[i] = live ? *reinterpret_cast<const uint4*>(row + col + 8 * l) : make_uint4(0u, 0u, 0u, 0u);
     }
     const bool turns = a.cos_t != nullptr, lower = turns && 8 * l < a.half, upper = turns && !lower && 8 * l < 2 * a.half;
     float c[8], sn[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) { c[i] = 1.f; sn[i] = 0.f; }
-    if (sub < hpw && (lower || upper)) {
+    if (lower || upper) {
         const int at = lower ? 8 * l : 8 * l - a.half;
         prep_load8(a.cos_t + (size_t)t * a.half + at, c);
         prep_load8(a.sin_t + (size_t)t * a.half + at, sn);
@@ -311,7 +311,7 @@ __global__ void __launch_bounds__(128) head_prep_heads_kernel(__nv_bfloat16* __r
 #pragma unroll
     for (int i = 0; i < HPG; ++i) {
         const int head = head0 + i * step;
-        bool live = sub < hpw && head < a.H + n_k + n_v;
+        bool live = head < a.H + n_k + n_v;
         const bool is_q = head < a.H, is_v = head >= a.H + n_k;
         if (live && !is_q) {
             if (slot >= a.pool_slots) { if (l == 0) oxr_report(a.status, OXR_BAD_SLOT, t); live = false; }
@@ -323,7 +323,7 @@ __global__ void __launch_bounds__(128) head_prep_heads_kernel(__nv_bfloat16* __r
         prep_unpack(raw[i], y);
         if (a.bias != nullptr && live && !is_v) {
             float b[8];
-            prep_load8(a.bias + (is_q ? 0 : a.H * a.DK) + h * a.DK + 8 * l, b);
+            prep_load8(a.bias + (is_q ? 0 : a.H * DK) + h * DK + 8 * l, b);
 #pragma unroll
             for (int k = 0; k < 8; ++k) y[k] += b[k];
         }
@@ -338,7 +338,9 @@ __global__ void __launch_bounds__(128) head_prep_heads_kernel(__nv_bfloat16* __r
             float sq = 0.f;
 #pragma unroll
             for (int k = 0; k < 8; ++k) sq = fmaf(y[k], y[k], sq);
-            const float inv = 1.f / sqrtf(prep_head_sum(sq, g0, lph) / (float)a.DK + a.eps);
+#pragma unroll
+            for (int o = LPH >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            const float inv = rsqrtf(sq * (1.f / (float)DK) + a.eps);
 #pragma unroll
             for (int k = 0; k < 8; ++k) y[k] = y[k] * inv * wn[k];
         }
@@ -353,14 +355,16 @@ __global__ void __launch_bounds__(128) head_prep_heads_kernel(__nv_bfloat16* __r
             float sq = 0.f;
 #pragma unroll
             for (int k = 0; k < 8; ++k) sq = fmaf(y[k], y[k], sq);
-            const float inv = 1.f / sqrtf(prep_head_sum(sq, g0, lph) / (float)a.DK + a.eps);
+#pragma unroll
+            for (int o = LPH >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            const float inv = rsqrtf(sq * (1.f / (float)DK) + a.eps);
 #pragma unroll
             for (int k = 0; k < 8; ++k) y[k] = y[k] * inv * wn[k];
         }
         if (live && !is_v) {
 #pragma unroll
             for (int k = 0; k < 8; ++k) y[k] *= f;
-            bf16* dst = is_q ? q_out + ((size_t)t * a.H + h) * a.DK : k_pool + ((long long)slot * a.KV + h) * a.DK;
+            bf16* dst = is_q ? q_out + ((size_t)t * a.H + h) * DK : k_pool + ((long long)slot * a.KV + h) * DK;
             *reinterpret_cast<uint4*>(dst + 8 * l) = prep_pack(y);
         }
     }
@@ -418,12 +422,13 @@ OXR_API int oxr_head_prep(void* q_out, void* k_pool, void* v_pool, const void* p
         const int per_block = 4 * hpw;
         dim3 vgrid(n_tokens, (heads + per_block - 1) / per_block);
         if (vgrid.y > 65535) return OXR_BAD_ARGUMENT;
-        const bool no_filter = taps == nullptr && n_tokens >= 64;
-        const int hpg = no_filter ? (heads >= 4 * per_block ? 4 : (heads >= 2 * per_block ? 2 : 1)) : 1;
-        if (hpg > 1) {
-            dim3 hgrid(n_tokens, (heads + per_block * hpg - 1) / (per_block * hpg));
-            if (hpg == 4) head_prep_heads_kernel<4><<<hgrid, 128, 0, stream>>>((__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)proj, a, lph, hpw);
-            else head_prep_heads_kernel<2><<<hgrid, 128, 0, stream>>>((__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)proj, a, lph, hpw);
+        if (taps == nullptr && n_tokens >= 64 && heads >= 2 * per_block && (lph == 8 || lph == 16)) {      // heads of 64 and of 128 entries
+            dim3 hgrid(n_tokens, (heads + 2 * per_block - 1) / (2 * per_block));
+#define OXR_PREP_HEADS(LPH) \
+    head_prep_heads_kernel<LPH, 2><<<hgrid, 128, 0, stream>>>((__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)proj, a)
+            if (lph == 8) OXR_PREP_HEADS(8);
+            else OXR_PREP_HEADS(16);
+#undef OXR_PREP_HEADS
             return oxr_launch_status();
         }
         head_prep_bf16x8_kernel<<<vgrid, 128, 0, stream>>>((__nv_bfloat16*)q_out, (__nv_bfloat16*)k_pool, (__nv_bfloat16*)v_pool, (const __nv_bfloat16*)proj, a, lph, hpw);
