@@ -19,7 +19,7 @@ class DeltaRule(Mixer):
 
         S_t = diag(w_t) S_(t-1) - (a_t * u_t) (u_t^T S_(t-1)) + k_t v_t^T        o_t = S_t^T r_t
 
-    (both terms read the old state). Then each head's o is divided by its root mean square, the heads side by side are multiplied by ``norm``
+    with everything on the right taken from S_(t-1). Then each head's o is divided by its root mean square, the heads side by side are multiplied by ``norm``
     (one weight per head and entry) and by ``sigmoid(W_g h)``, then ``W_o``. r, k, v and the gate are one product; ``W_a`` and ``W_w1`` are a second
     one whose result stays fp32, like that of ``W_w2`` and everything else that enters the recurrence behind the projections. Per request the
     mixer keeps one fp32 state row: S transposed, ``[heads, values, keys]``; zero for a new request, carried from step to step whatever the

@@ -89,7 +89,7 @@ SINGLE = {
     "differential_window_of_one": CFG([D(size=1)]),
     "differential_window_beyond_the_prompt": CFG([D(size=500)]),
     "differential_odd_sizes": CFG([D(heads=3, kv_heads=1, dim=7, vdim=11, size=5, diff=0.8)], width=39),
-    "differential_tma_sizes": CFG([D(heads=4, kv_heads=2, dim=32, vdim=64, size=21, scale=0.3)], width=64),
+    "differential_tma_sizes": CFG([D(heads=6, kv_heads=3, dim=32, vdim=64, size=21, scale=0.3)], width=64),
     "pair_alone": CFG([P()]),
     "pair_equal_sizes_all_rotated": CFG([P(heads=6, kv_heads=3, dim=32, vdim=32, rot=32, size=17, scale=0.2, r_heads=2, r_dim=16)], width=64),
     "pair_two_rotated_entries": CFG([P(rot=2, base=5.0, size=3)]),
@@ -456,7 +456,7 @@ WINDOW = 21
 
 # the marked key: far back (outside the window), just outside and just inside it for the last token, on a page's first and last row, the query itself
 @pytest.mark.parametrize("mark", [0, 7, 8, 129 - WINDOW, 130 - WINDOW, 119, 120, 128, 129])
-@pytest.mark.parametrize("dtype,H,G,D,DV", [("float32", 3, 1, 10, 24), ("bfloat16", 4, 2, 32, 64), ("bfloat16", 2, 2, 24, 16), ("bfloat16", 4, 1, 64, 128)])
+@pytest.mark.parametrize("dtype,H,G,D,DV", [("float32", 3, 1, 10, 24), ("bfloat16", 6, 2, 32, 64), ("bfloat16", 2, 2, 24, 16), ("bfloat16", 4, 1, 64, 128)])
 def test_marked_keys_inside_and_outside_the_window_of_both_maps(dtype, H, G, D, DV, mark):
     marked_case(dtype, H, G, D, DV, WINDOW, [70, 1, 5, 2], [130, 130, 130, 2], [mark, mark, mark, 0])
     marked_case(dtype, H, G, D, DV, 0, [70, 1, 5, 2], [130, 130, 130, 2], [mark, mark, mark, 0])

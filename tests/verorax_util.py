@@ -57,7 +57,7 @@ MODEL_B = model_config([*_B, again(_B, 0), latent(heads=1, dim=24, rot_dim=2, vd
 # every attention layer has sizes that the tensor-core kernels take in bfloat16, and its only router stands in the last layer, where a choice
 # that a rounding step turns over spoils one row and no later one
 _C = [latent(heads=4, dim=32, rot_dim=16, vdim=32, kv_rank=48, q_rank=64, base=500.0, scale=0.2, mlp=dense(ff=48)),
-      differential(heads=6, kv_heads=2, dim=32, vdim=64, size=33, diff=0.5, scale=0.3, mlp=dense(ff=32)),
+      differential(heads=6, kv_heads=2, dim=32, vdim=64, size=33, diff=0.45, scale=0.3, mlp=dense(ff=32)),
       paired(heads=4, kv_heads=1, dim=128, vdim=128, size=50, rot=64, base=1e3, scale=0.1, r_heads=2, r_dim=64, rank=8, mlp=dense(ff=40))]
 MODEL_C = model_config([*_C, again(_C, 2), differential(heads=4, kv_heads=4, dim=16, vdim=48, size=17, diff=0.1, scale=0.4), again(_C, 0),
                         latent(heads=8, dim=64, rot_dim=32, vdim=64, kv_rank=96, q_rank=32, base=1e4, scale=0.15, mlp=moe(ff=32, experts=4, identity=2, top=3))],
