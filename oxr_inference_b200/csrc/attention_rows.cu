@@ -211,9 +211,9 @@ __global__ void latent_prep_kernel(T* __restrict__ pool, long long slot_stride, 
         }
 }
 
-// The same for bf16 and half-split pairs, everything whole 16-byte words (rank, rot, half, strides and offsets multiples of 8; rot == 2 half). Warp 0
-// writes the cache row; every thread then takes one pair of words (w and w + half / 8 of a rotated part) and walks over the heads with its
-// angles in registers.
+// The same for bf16, everything whole 16-byte words (rank, rot, strides and offsets multiples of 8; with HALVES half, too; rot == 2 half). Warp 0
+// writes the cache row; every thread then takes one piece of a rotated part (HALVES: the words w and w + half / 8; else the four neighbouring
+// pairs of word w) and walks over the heads with the piece's angles in registers.
 __device__ __forceinline__ void lp_unpack(const uint4& v, float (&out)[8]) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
 #pragma unroll
@@ -229,9 +229,24 @@ __device__ __forceinline__ uint4 lp_pack(const float (&v)[8]) {
     for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
     return out;
 }
-__device__ __forceinline__ void lp_load8(const float* p, float (&out)[8]) {
+__device__ __forceinline__ void lp_load(const float* p, float (&out)[8]) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
     out[0] = a.x; out[1] = a.y; out[2] = a.z; out[3] = a.w; out[4] = b.x; out[5] = b.y; out[6] = b.z; out[7] = b.w;
+}
+__device__ __forceinline__ void lp_load(const float* p, float (&out)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    out[0] = a.x; out[1] = a.y; out[2] = a.z; out[3] = a.w;
+}
+// the four pairs of neighbours in one word
+__device__ __forceinline__ void lp_turn(__nv_bfloat16* dst, const __nv_bfloat16* src, int, const float (&c)[4], const float (&s)[4]) {
+    float x[8], o[8];
+    lp_unpack(*reinterpret_cast<const uint4*>(src), x);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        o[2 * i] = x[2 * i] * c[i] - x[2 * i + 1] * s[i];
+        o[2 * i + 1] = x[2 * i + 1] * c[i] + x[2 * i] * s[i];
+    }
+    *reinterpret_cast<uint4*>(dst) = lp_pack(o);
 }
 // (u, v) -> (u cos - v sin, v cos + u sin) for the words at p and p + half
 __device__ __forceinline__ void lp_turn(__nv_bfloat16* dst, const __nv_bfloat16* src, int half, const float (&c)[8], const float (&s)[8]) {
@@ -247,13 +262,15 @@ __device__ __forceinline__ void lp_turn(__nv_bfloat16* dst, const __nv_bfloat16*
     *reinterpret_cast<uint4*>(dst + half) = lp_pack(b);
 }
 
+template <bool HALVES>
 __global__ void __launch_bounds__(128) latent_prep_words_kernel(__nv_bfloat16* __restrict__ pool, long long slot_stride, long long pool_slots,
                                                                 const __nv_bfloat16* __restrict__ down, int down_stride, int rank,
                                                                 const float* __restrict__ weight, float eps, const __nv_bfloat16* q, int heads,
                                                                 int q_head_dim, int q_rot0, __nv_bfloat16* q_out, int qo_head_dim, int qo_rot0,
                                                                 const float* __restrict__ cos_t, const float* __restrict__ sin_t, int half,
                                                                 const int* __restrict__ slots, int* status) {
-    const int t = blockIdx.x, lane = threadIdx.x & 31, slot = slots[t], per = half / 8;     // words of half a rotated part
+    constexpr int A = HALVES ? 8 : 4;                                                       // angles of a piece
+    const int t = blockIdx.x, lane = threadIdx.x & 31, slot = slots[t], per = half / A;     // pieces of a rotated part
     const __nv_bfloat16* row = down + (size_t)t * down_stride;
     const float* ct = cos_t + (size_t)t * half;
     const float* st = sin_t + (size_t)t * half;
@@ -272,24 +289,24 @@ __global__ void __launch_bounds__(128) latent_prep_words_kernel(__nv_bfloat16* _
             for (int i = lane; i < rank / 8; i += 32) {
                 float w[8];
                 lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), x);
-                lp_load8(weight + 8 * i, w);
+                lp_load(weight + 8 * i, w);
 #pragma unroll
                 for (int k = 0; k < 8; ++k) x[k] = x[k] * inv * w[k];
                 *reinterpret_cast<uint4*>(dst + 8 * i) = lp_pack(x);
             }
             for (int i = lane; i < per; i += 32) {
-                float c[8], s[8];
-                lp_load8(ct + 8 * i, c);
-                lp_load8(st + 8 * i, s);
+                float c[A], s[A];
+                lp_load(ct + A * i, c);
+                lp_load(st + A * i, s);
                 lp_turn(dst + rank + 8 * i, row + rank + 8 * i, half, c, s);
             }
         }
     }
-    const int w = threadIdx.x % per, stride = blockDim.x / per;      // one word per thread; stride threads with the same word share the heads
+    const int w = threadIdx.x % per, stride = blockDim.x / per;      // one piece per thread; stride threads with the same piece share the heads
     if ((int)threadIdx.x < stride * per) {
-        float c[8], s[8];
-        lp_load8(ct + 8 * w, c);
-        lp_load8(st + 8 * w, s);
+        float c[A], s[A];
+        lp_load(ct + A * w, c);
+        lp_load(st + A * w, s);
         for (int h = threadIdx.x / per; h < heads; h += stride)
             lp_turn(q_out + ((size_t)t * heads + h) * qo_head_dim + qo_rot0 + 8 * w, q + ((size_t)t * heads + h) * q_head_dim + q_rot0 + 8 * w, half, c, s);
     }
@@ -326,7 +343,7 @@ __global__ void __launch_bounds__(128) cols_rms_norm_words_kernel(__nv_bfloat16*
         } else {
             lp_unpack(*reinterpret_cast<const uint4*>(row + 8 * i), y);
         }
-        lp_load8(weight + 8 * i, w);
+        lp_load(weight + 8 * i, w);
 #pragma unroll
         for (int e = 0; e < 8; ++e) y[e] = y[e] * inv * w[e];
         *reinterpret_cast<uint4*>(out + (size_t)blockIdx.x * width + 8 * i) = lp_pack(y);
@@ -338,12 +355,13 @@ OXR_API int oxr_latent_prep(void* pool, long long slot_stride, long long pool_sl
                             const float* sin_t, int half, int halves, const int* slots, int n_tokens, int dtype, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (rank <= 0 || down_stride < rank + rot || rot < 0 || 2 * half > rot || q_rot0 + rot > q_head_dim || qo_rot0 + rot > qo_head_dim) return OXR_BAD_ARGUMENT;
-    if (dtype == 1 && halves && half > 0 && half % 8 == 0 && half <= 1024 && rot == 2 * half && rank % 8 == 0 && slot_stride % 8 == 0 && down_stride % 8 == 0 &&
+    if (dtype == 1 && half > 0 && half % (halves ? 8 : 4) == 0 && half <= (halves ? 1024 : 512) && rot == 2 * half && rank % 8 == 0 && slot_stride % 8 == 0 && down_stride % 8 == 0 &&
         q_head_dim % 8 == 0 && q_rot0 % 8 == 0 && qo_head_dim % 8 == 0 && qo_rot0 % 8 == 0 && (uintptr_t)pool % 16 == 0 && (uintptr_t)down % 16 == 0 &&
         (uintptr_t)q % 16 == 0 && (uintptr_t)q_out % 16 == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)cos_t % 16 == 0 && (uintptr_t)sin_t % 16 == 0) {
-        latent_prep_words_kernel<<<n_tokens, 128, 0, stream>>>((__nv_bfloat16*)pool, slot_stride, pool_slots, (const __nv_bfloat16*)down, down_stride, rank, weight,
-                                                              eps, (const __nv_bfloat16*)q, heads, q_head_dim, q_rot0, (__nv_bfloat16*)q_out, qo_head_dim, qo_rot0,
-                                                              cos_t, sin_t, half, slots, status);
+        const auto kernel = halves ? latent_prep_words_kernel<true> : latent_prep_words_kernel<false>;
+        kernel<<<n_tokens, 128, 0, stream>>>((__nv_bfloat16*)pool, slot_stride, pool_slots, (const __nv_bfloat16*)down, down_stride, rank, weight, eps,
+                                             (const __nv_bfloat16*)q, heads, q_head_dim, q_rot0, (__nv_bfloat16*)q_out, qo_head_dim, qo_rot0, cos_t, sin_t, half,
+                                             slots, status);
         return oxr_launch_status();
     }
     if (dtype == 0)

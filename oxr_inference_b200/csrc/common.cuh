@@ -114,7 +114,7 @@ inline int oxr_chain_kernels = 0;   // one per library: set through oxr_set_chai
 
 // What the gated epilogue of a product computes from a gate sum g and an up sum u. kind 0: silu(g) * u. kind 1: with
 // g' = min(g, limit) and u' = clamp(u, -limit, limit): g' * sigmoid(alpha g') * (u' + 1). kind 3: gelu(g) * u with the tanh form of
-// gelu (kind 2 is a plain product's relu(x)^2, which has no up sum). The launchers of the gated products hand
+// gelu (kind 2 is a plain product's relu(x)^2, which has no up sum: RELU2_FORM). The launchers of the gated products hand
 // the library's current form to their kernels by value; oxr_set_gate_form() sets it (before each gated call).
 struct GateForm {
     int kind;
@@ -122,6 +122,7 @@ struct GateForm {
     float limit;
 };
 inline GateForm oxr_gate_form = {0, 1.f, 0.f};
+constexpr GateForm PLAIN_FORM = {0, 1.f, 0.f}, RELU2_FORM = {2, 0.f, 0.f};
 __device__ __forceinline__ float gate_apply(const GateForm& f, float g, float u) {
     if (f.kind == 1) {
         g = fminf(g, f.limit);

@@ -6,7 +6,8 @@
 // tie); their weights are their s divided by the sum of the chosen s (+ 1e-20), times `scale`. All of it in fp32.
 // Variants, each an argument: scores that are the softmax of z over all experts instead of sigmoids (score_kind 1); a group's
 // score that is its largest s instead of the sum of its two largest (group_kind 1); weights that are the chosen s themselves,
-// times `scale`, not divided by their sum (renorm 0); choice scores s + correction[e] (groups and experts are then picked by these, the
+// times `scale`, not divided by their sum (renorm 0); the logits themselves as choice scores and exp(z - max z) as s (score_kind 2, with renorm:
+// the weights are then the softmax over the chosen logits); a bias per expert added to the logits first; choice scores s + correction[e] (groups and experts are then picked by these, the
 // weights stay those of s); and identity experts: of the E scored experts the last E - real return their input, so that they need no product:
 // the token's weights for them are added up in `kept` [tokens], and the dense row has the real experts' columns only.
 //
@@ -24,17 +25,21 @@ constexpr int ROUTE_MAX_GROUPS = 64;
 
 __global__ void route_kernel(float* __restrict__ gate, int* __restrict__ ids, float* __restrict__ wts, const float* __restrict__ z, int n_tokens,
                              int E, int top, int groups, int keep, float scale, int score_kind, int group_kind, int renorm, const float* __restrict__ correction,
-                             int real, float* __restrict__ kept) {
+                             int real, float* __restrict__ kept, const float* __restrict__ bias) {
     const int t = blockIdx.x * blockDim.x + threadIdx.x;
     if (t >= n_tokens) return;
-    const float* zr = z + (size_t)t * E;
+    auto logit = [&](int e) { return bias != nullptr ? z[(size_t)t * E + e] + bias[e] : z[(size_t)t * E + e]; };
     float zmax = -INFINITY, den = 0.f;
-    if (score_kind == 1) {
-        for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, zr[e]);
-        for (int e = 0; e < E; ++e) den += expf(zr[e] - zmax);
+    if (score_kind != 0) {
+        for (int e = 0; e < E; ++e) zmax = fmaxf(zmax, logit(e));
+        for (int e = 0; e < E; ++e) den += expf(logit(e) - zmax);
     }
-    auto score_of = [&](int e) { return score_kind == 1 ? expf(zr[e] - zmax) / den : 1.f / (1.f + expf(-zr[e])); };
-    auto choice_of = [&](int e) { return correction != nullptr ? score_of(e) + correction[e] : score_of(e); };
+    if (score_kind == 2) den = 1.f;
+    auto score_of = [&](int e) { return score_kind != 0 ? expf(logit(e) - zmax) / den : 1.f / (1.f + expf(-logit(e))); };
+    auto choice_of = [&](int e) {
+        if (score_kind == 2) return logit(e);
+        return correction != nullptr ? score_of(e) + correction[e] : score_of(e);
+    };
     unsigned long long allowed = ~0ull;        // one bit per group
     const int per = E / groups;
     if (groups > 1 && keep < groups) {
@@ -106,7 +111,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& idx) {
 __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gate, int* __restrict__ ids, float* __restrict__ wts, const float* __restrict__ z,
                                                         int n_tokens, int E, int top, int groups, int keep, float scale, int score_kind,
                                                         int group_kind, int renorm, const float* __restrict__ correction, int real,
-                                                        float* __restrict__ kept) {
+                                                        float* __restrict__ kept, const float* __restrict__ bias) {
     __shared__ float sc[4][ROUTE_WARP_MAX_E], ch[4][ROUTE_WARP_MAX_E];     // scores, choice scores
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * 4 + warp;
@@ -114,17 +119,19 @@ __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gat
     float* s = sc[warp];
     float* cs = ch[warp];
     const int per = E / groups;
-    if (score_kind == 1) {
+    auto logit = [&](int e) { return bias != nullptr ? z[(size_t)t * E + e] + bias[e] : z[(size_t)t * E + e]; };
+    if (score_kind != 0) {
         float zmax = -INFINITY, den = 0.f;
-        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[(size_t)t * E + e]);
+        for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, logit(e));
         zmax = warp_max(zmax);
-        for (int e = lane; e < E; e += 32) { s[e] = expf(z[(size_t)t * E + e] - zmax); den += s[e]; }
+        for (int e = lane; e < E; e += 32) { s[e] = expf(logit(e) - zmax); den += s[e]; }
         den = warp_sum(den);
-        for (int e = lane; e < E; e += 32) s[e] = s[e] / den;
+        if (score_kind == 1)
+            for (int e = lane; e < E; e += 32) s[e] = s[e] / den;
     } else {
-        for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-z[(size_t)t * E + e]));
+        for (int e = lane; e < E; e += 32) s[e] = 1.f / (1.f + expf(-logit(e)));
     }
-    for (int e = lane; e < E; e += 32) cs[e] = correction != nullptr ? s[e] + correction[e] : s[e];     // each lane reads what it wrote
+    for (int e = lane; e < E; e += 32) cs[e] = score_kind == 2 ? logit(e) : correction != nullptr ? s[e] + correction[e] : s[e];     // each lane reads what it wrote
     __syncwarp();
     unsigned allowed = 0xffffffffu;            // one bit per group
     if (groups > 1 && keep < groups) {
@@ -184,15 +191,15 @@ __global__ void __launch_bounds__(128) route_warp_kernel(float* __restrict__ gat
 }
 
 OXR_API int oxr_route(float* gate, int* ids, float* wts, const float* z, int n_tokens, int E, int top, int groups, int keep, float scale,
-                      int score_kind, int group_kind, int renorm, const float* correction, int real, float* kept, cudaStream_t stream) {
+                      int score_kind, int group_kind, int renorm, const float* correction, int real, float* kept, const float* bias, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (real <= 0 || real > E || (real < E && kept == nullptr) || E <= 0 || top <= 0 || top > E || top > ROUTE_MAX_TOP || groups <= 0 || groups > ROUTE_MAX_GROUPS || E % groups || keep <= 0 || keep > groups ||
-        top > keep * (E / groups) || score_kind < 0 || score_kind > 1 || group_kind < 0 || group_kind > 1)
+        top > keep * (E / groups) || score_kind < 0 || score_kind > 2 || (score_kind == 2 && (!renorm || correction != nullptr)) || group_kind < 0 || group_kind > 1)
         return OXR_BAD_ARGUMENT;
     if (E <= ROUTE_WARP_MAX_E && groups <= 32)
-        route_warp_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept);
+        route_warp_kernel<<<(n_tokens + 3) / 4, 128, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept, bias);
     else
-        route_kernel<<<(n_tokens + 63) / 64, 64, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept);
+        route_kernel<<<(n_tokens + 63) / 64, 64, 0, stream>>>(gate, ids, wts, z, n_tokens, E, top, groups, keep, scale, score_kind, group_kind, renorm, correction, real, kept, bias);
     return oxr_launch_status();
 }
 

@@ -300,6 +300,7 @@ gemm_stream_kernel(TO* __restrict__ C, const __nv_bfloat16* __restrict__ X, cons
 #pragma unroll
                     for (int w = 0; w < ST_WARPS; ++w) s += partial[(w * 16 + r) * PW + m];
                     if constexpr (SCALED) s *= s_inv[m];
+                    if (gate.kind == 2) { s = fmaxf(s, 0.f); s *= s; }   // the plain product's optional activation
                     C[(size_t)m * N + n0 + r] = Num<TO>::from_f32(s);
                 }
             }
@@ -330,7 +331,7 @@ gemm_stream_kernel(TO* __restrict__ C, const __nv_bfloat16* __restrict__ X, cons
 }
 
 template <int TILES, typename TO, bool GATED, bool ADD = false, bool SCALED = false>
-int launch_stream(void* C, const void* X, const void* W, int M, int N, int K, int* status, cudaStream_t stream, FuseArgs fa = FuseArgs{}) {
+int launch_stream(void* C, const void* X, const void* W, int M, int N, int K, int* status, cudaStream_t stream, FuseArgs fa = FuseArgs{}, int act = 0) {
     static int sms = 0, stages = 0;
     static size_t smem = 0;
     if (sms == 0) {
@@ -353,19 +354,23 @@ int launch_stream(void* C, const void* X, const void* W, int M, int N, int K, in
     const int groups = (N + 15) / 16;
     const int blocks = groups < sms ? groups : sms;
     oxr_launch(gemm_stream_kernel<TILES, TO, GATED, ADD, SCALED>, dim3(blocks), dim3(ST_THREADS), smem, stream, true,
-               (TO*)C, (const __nv_bfloat16*)X, (const __nv_bfloat16*)W, M, N, K, stages, status, fa, oxr_gate_form);
+               (TO*)C, (const __nv_bfloat16*)X, (const __nv_bfloat16*)W, M, N, K, stages, status, fa, act == 1 ? RELU2_FORM : (GATED ? oxr_gate_form : PLAIN_FORM));
     return oxr_launch_status();
 }
 }  // namespace
 
-// out_dtype: 0 = float32, 1 = bfloat16. Requires M <= 16, K % 8 == 0 and 16-byte aligned X and W.
-OXR_API int oxr_gemm_stream_bf16(void* C, const void* X, const void* W, int M, int N, int K, int out_dtype, int* status,
+// out_dtype: 0 = float32, 1 = bfloat16. Requires M <= 16, K % 8 == 0 and 16-byte aligned X and W. act 1: the output is relu(x)^2 of the fp32 sums.
+OXR_API int oxr_gemm_stream_bf16(void* C, const void* X, const void* W, int M, int N, int K, int out_dtype, int act, int* status,
                                  cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
+    if (act != 0 && act != 1) return OXR_BAD_ARGUMENT;
     if (M > 16 || K <= 0 || K % 8 != 0 || (uintptr_t)X % 16 != 0 || (uintptr_t)W % 16 != 0) return OXR_BAD_ARGUMENT;
     using bf = __nv_bfloat16;
-    if (out_dtype == 0) return M <= 8 ? launch_stream<1, float, false>(C, X, W, M, N, K, status, stream) : launch_stream<2, float, false>(C, X, W, M, N, K, status, stream);
-    if (out_dtype == 1) return M <= 8 ? launch_stream<1, bf, false>(C, X, W, M, N, K, status, stream) : launch_stream<2, bf, false>(C, X, W, M, N, K, status, stream);
+    const FuseArgs none{};
+    if (out_dtype == 0)
+        return M <= 8 ? launch_stream<1, float, false>(C, X, W, M, N, K, status, stream, none, act) : launch_stream<2, float, false>(C, X, W, M, N, K, status, stream, none, act);
+    if (out_dtype == 1)
+        return M <= 8 ? launch_stream<1, bf, false>(C, X, W, M, N, K, status, stream, none, act) : launch_stream<2, bf, false>(C, X, W, M, N, K, status, stream, none, act);
     return OXR_BAD_ARGUMENT;
 }
 

@@ -221,13 +221,7 @@ gemm_tcgen05_kernel(TO* __restrict__ C, const __grid_constant__ CUtensorMap map_
                     } else if (n0 + c0 < N) {
                         if constexpr (GATED) store_row_piece_gated<TO>(C + (size_t)row * (N / 2) + (n0 + c0) / 2, v, count, n0 + c0, N, gate);
                         else {
-                            if (gate.kind == 2) {   // the plain product's optional activation: relu(x)^2 of the fp32 sums
-#pragma unroll
-                                for (int j = 0; j < 32; ++j) {
-                                    const float f = fmaxf(__uint_as_float(v[j]), 0.f);
-                                    v[j] = __float_as_uint(f * f);
-                                }
-                            }
+                            if (gate.kind == 2) relu2_piece(v);   // the plain product's optional activation
                             store_row_piece<TO>(C + (size_t)row * N + n0 + c0, v, count, n0 + c0, N);
                         }
                     }
@@ -333,7 +327,7 @@ int launch(void* C, const void* X, const void* W, int M, int N, int K, int bn, i
     while (tmem_cols < 2 * bn) tmem_cols *= 2;
     dim3 grid((unsigned)(units < num_sms ? units : num_sms));   // one block per SM (its shared memory fills the SM)
     oxr_launch(gemm_tcgen05_kernel<TO, SPLIT, GATED>, grid, dim3(TC_THREADS), SMEM_BYTES, stream, true, (TO*)C, map_x, map_w, M, N, K, bn,
-               stages, tmem_cols, (int)tiles, splits, partial, tickets, status, act == 1 ? GateForm{2, 0.f, 0.f} : (GATED ? oxr_gate_form : GateForm{0, 1.f, 0.f}),
+               stages, tmem_cols, (int)tiles, splits, partial, tickets, status, act == 1 ? RELU2_FORM : (GATED ? oxr_gate_form : PLAIN_FORM),
                tile_group);
     return oxr_launch_status();
 }
@@ -343,10 +337,11 @@ int launch(void* C, const void* X, const void* W, int M, int N, int K, int bn, i
 // tile_n: columns of the output per tile, a multiple of 16 from 16 to 256.
 // splits > 1 deals the 64-wide k steps out to that many shares per tile (at most as many as steps); `partial` then
 // holds splits * tiles * 128 * tile_n floats (tiles = ceil(M / 128) * ceil(N / tile_n)) and `tickets` one zeroed
-// counter per tile, which the kernel leaves zeroed.
+// counter per tile, which the kernel leaves zeroed. act 1 (without shares of k): the output is relu(x)^2 of the fp32 sums.
 OXR_API int oxr_gemm_tcgen05_bf16(void* C, const void* X, const void* W, int M, int N, int K, int out_dtype, int tile_n, int splits,
-                                  float* partial, unsigned int* tickets, int* status, cudaStream_t stream) {
+                                  float* partial, unsigned int* tickets, int act, int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
+    if (act != 0 && (act != 1 || splits > 1)) return OXR_BAD_ARGUMENT;
     if (K <= 0 || K % 8 != 0 || (uintptr_t)X % 16 != 0 || (uintptr_t)W % 16 != 0) return OXR_BAD_ARGUMENT;
     if (tile_n < 16 || tile_n > MAX_BN || tile_n % 16 != 0) return OXR_BAD_ARGUMENT;
     if (splits > 1) {
@@ -355,8 +350,8 @@ OXR_API int oxr_gemm_tcgen05_bf16(void* C, const void* X, const void* W, int M, 
         if (out_dtype == 0) return launch<float, true>(C, X, W, M, N, K, tile_n, splits, partial, tickets, status, stream);
         return OXR_BAD_ARGUMENT;
     }
-    if (out_dtype == 1) return launch<__nv_bfloat16, false>(C, X, W, M, N, K, tile_n, 1, nullptr, nullptr, status, stream);
-    if (out_dtype == 0) return launch<float, false>(C, X, W, M, N, K, tile_n, 1, nullptr, nullptr, status, stream);
+    if (out_dtype == 1) return launch<__nv_bfloat16, false>(C, X, W, M, N, K, tile_n, 1, nullptr, nullptr, status, stream, 1, nullptr, act);
+    if (out_dtype == 0) return launch<float, false>(C, X, W, M, N, K, tile_n, 1, nullptr, nullptr, status, stream, 1, nullptr, act);
     return OXR_BAD_ARGUMENT;
 }
 

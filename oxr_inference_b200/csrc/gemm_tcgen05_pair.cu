@@ -200,7 +200,10 @@ gemm_tcgen05_pair_kernel(TO* __restrict__ C, const __grid_constant__ CUtensorMap
                 else tmem_ld_32x16(acc_addr + (uint32_t)c0, v);
                 if (row < M && n0 + c0 < N) {
                     if constexpr (GATED) store_row_piece_gated<TO>(C + (size_t)row * (N / 2) + (n0 + c0) / 2, v, count, n0 + c0, N, gate);
-                    else store_row_piece<TO>(C + (size_t)row * N + n0 + c0, v, count, n0 + c0, N);
+                    else {
+                        if (gate.kind == 2) relu2_piece(v);   // the plain product's optional activation
+                        store_row_piece<TO>(C + (size_t)row * N + n0 + c0, v, count, n0 + c0, N);
+                    }
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -217,7 +220,7 @@ gemm_tcgen05_pair_kernel(TO* __restrict__ C, const __grid_constant__ CUtensorMap
 }
 
 template <typename TO, bool GATED = false>
-int launch_pair(void* C, const void* X, const void* W, int M, int N, int K, int bn, int* status, cudaStream_t stream) {
+int launch_pair(void* C, const void* X, const void* W, int M, int N, int K, int bn, int* status, cudaStream_t stream, int act = 0) {
     static int max_pairs = 0;   // per instantiation
     if (max_pairs == 0) {
         cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<TO, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
@@ -253,20 +256,21 @@ int launch_pair(void* C, const void* X, const void* W, int M, int N, int K, int 
     while (tmem_cols < 2 * bn) tmem_cols *= 2;
     const unsigned pairs = (unsigned)(tiles < max_pairs ? tiles : max_pairs);
     oxr_launch(gemm_tcgen05_pair_kernel<TO, GATED>, dim3(2 * pairs), dim3(PAIR_THREADS), SMEM_BYTES, stream, true, (TO*)C, map_x, map_w, M, N, K,
-               bn, stages, tmem_cols, (int)tiles, status, oxr_gate_form);
+               bn, stages, tmem_cols, (int)tiles, status, act == 1 ? RELU2_FORM : (GATED ? oxr_gate_form : PLAIN_FORM));
     return oxr_launch_status();
 }
 }  // namespace
 
 // out_dtype: 0 = float32, 1 = bfloat16. Requires K % 8 == 0 and 16-byte aligned X, W. tile_n: columns of the output
-// per pair of blocks, a multiple of 32 from 32 to 256 (each block stages half of them).
-OXR_API int oxr_gemm_tcgen05_pair_bf16(void* C, const void* X, const void* W, int M, int N, int K, int out_dtype, int tile_n, int* status,
+// per pair of blocks, a multiple of 32 from 32 to 256 (each block stages half of them). act 1: the output is relu(x)^2 of the fp32 sums.
+OXR_API int oxr_gemm_tcgen05_pair_bf16(void* C, const void* X, const void* W, int M, int N, int K, int out_dtype, int tile_n, int act, int* status,
                                        cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
+    if (act != 0 && act != 1) return OXR_BAD_ARGUMENT;
     if (K <= 0 || K % 8 != 0 || (uintptr_t)X % 16 != 0 || (uintptr_t)W % 16 != 0) return OXR_BAD_ARGUMENT;
     if (tile_n < 32 || tile_n > MAX_BN || tile_n % 32 != 0) return OXR_BAD_ARGUMENT;
-    if (out_dtype == 1) return launch_pair<__nv_bfloat16>(C, X, W, M, N, K, tile_n, status, stream);
-    if (out_dtype == 0) return launch_pair<float>(C, X, W, M, N, K, tile_n, status, stream);
+    if (out_dtype == 1) return launch_pair<__nv_bfloat16>(C, X, W, M, N, K, tile_n, status, stream, act);
+    if (out_dtype == 0) return launch_pair<float>(C, X, W, M, N, K, tile_n, status, stream, act);
     return OXR_BAD_ARGUMENT;
 }
 

@@ -208,15 +208,15 @@ __global__ void gelu_glu_kernel(T* __restrict__ out, const T* __restrict__ gate_
 }
 
 // ---------------------------------------------------------------------------------------------- rotary angles
-// cos/sin [tokens, half] of position * freq[i], the product and the functions in fp64, rounded once to fp32.
+// cos/sin [tokens, half] of position * freq[i], times `magnitude`: products and functions in fp64, rounded once to fp32.
 __global__ void rotary_angles_kernel(float* __restrict__ cos_out, float* __restrict__ sin_out, const int* __restrict__ positions,
-                                     const double* __restrict__ freq, int half, int total) {
+                                     const double* __restrict__ freq, double magnitude, int half, int total) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     double s, c;
     sincos((double)positions[i / half] * freq[i % half], &s, &c);
-    cos_out[i] = (float)c;
-    sin_out[i] = (float)s;
+    cos_out[i] = (float)(c * magnitude);
+    sin_out[i] = (float)(s * magnitude);
 }
 
 // ---------------------------------------------------------------------------------------------- launchers
@@ -302,10 +302,10 @@ OXR_API int oxr_gelu_glu(void* out, const void* gate_up, int n, int inter, int i
     return oxr_launch_status();
 }
 
-OXR_API int oxr_rotary_angles(float* cos_out, float* sin_out, const int* positions, const double* freq, int n, int half, cudaStream_t stream_) {
+OXR_API int oxr_rotary_angles(float* cos_out, float* sin_out, const int* positions, const double* freq, double magnitude, int n, int half, cudaStream_t stream_) {
     if (n <= 0 || half <= 0) return 0;
     const int total = n * half;
-    rotary_angles_kernel<<<(total + 127) / 128, 128, 0, stream_>>>(cos_out, sin_out, positions, freq, half, total);
+    rotary_angles_kernel<<<(total + 127) / 128, 128, 0, stream_>>>(cos_out, sin_out, positions, freq, magnitude, half, total);
     return oxr_launch_status();
 }
 

@@ -100,6 +100,14 @@ __device__ __forceinline__ void store_row_piece(TO* dst, const uint32_t (&v)[32]
     }
 }
 
+// relu(x)^2 of a piece of a plain product's fp32 sums
+__device__ __forceinline__ void relu2_piece(uint32_t (&v)[32]) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+        const float f = fmaxf(__uint_as_float(v[j]), 0.f);
+        v[j] = __float_as_uint(f * f);
+    }
+}
 
 // The same piece of a product whose columns alternate in groups of 8 between a gate and an up projection (columns
 // 16j .. 16j+7 gate 8j .. 8j+7, 16j+8 .. 16j+15 the matching up values; col0 a multiple of 16): writes

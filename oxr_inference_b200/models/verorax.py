@@ -20,7 +20,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Mapping
 
-from oxr_inference_b200.config.fields import need, nonneg_int, number, pos_int
+from oxr_inference_b200.config.fields import head_counts, need, nonneg_int, number, pos_int, weights_owner
 from oxr_inference_b200.config.model_config import ConfigError
 from oxr_inference_b200.config.registry import Architecture, register_architecture
 from oxr_inference_b200.parts.spec import LayerSpec, ModelSpec, PartSpec, ScheduleEntry
@@ -64,7 +64,7 @@ class VeroraxConfig:
             mlp = entry.get("mlp")
             if mlp is not None and need(mlp, "kind", where + ".mlp") not in _FEED_FORWARDS:
                 raise ConfigError(f"config.json: {where}.mlp.kind {mlp['kind']!r} is not one of {sorted(_FEED_FORWARDS)}")
-            layers.append(VeroraxLayer(kind, dict(need(entry, "mixer", where)), dict(mlp) if mlp is not None else None, _owner(listed, i)))
+            layers.append(VeroraxLayer(kind, dict(need(entry, "mixer", where)), dict(mlp) if mlp is not None else None, weights_owner(listed, i)))
         for i, layer in enumerate(layers):
             theirs = layers[layer.owner]
             if (layer.type, layer.mixer, layer.mlp) != (theirs.type, theirs.mixer, theirs.mlp):
@@ -81,27 +81,7 @@ class VeroraxConfig:
         return config
 
 
-def _owner(listed: list, i: int) -> int:
-    """Follow ``weights_of`` from layer i to the layer that has tensors."""
-    seen = {i}
-    at = i
-    while isinstance(listed[at], Mapping) and listed[at].get("weights_of") is not None:
-        j = listed[at]["weights_of"]
-        if isinstance(j, bool) or not isinstance(j, int) or not 0 <= j < len(listed) or j in seen:
-            raise ConfigError(f"config.json: layers[{at}].weights_of must name another layer that has tensors, got {j!r}")
-        seen.add(j)
-        at = j
-    return at
-
-
 # ---- the pieces of a mixer entry
-def _heads(m: Mapping[str, Any], where: str) -> dict[str, int]:
-    out = {"num_heads": pos_int(m, "heads", where), "num_kv_heads": pos_int(m, "kv_heads", where)}
-    if out["num_heads"] % out["num_kv_heads"]:
-        raise ConfigError(f"config.json: {where}: {out['num_heads']} heads are not a multiple of {out['num_kv_heads']} kv_heads")
-    return out
-
-
 def _rotation(m: Mapping[str, Any], where: str, entries: int) -> PartSpec | None:
     """The ``rot`` entry of a mixer as a half-split rotation within ``entries`` entries, None without one."""
     rot = m.get("rot")
@@ -136,7 +116,7 @@ def _latent(c: VeroraxConfig, i: int, shapes) -> tuple[PartSpec, PartSpec | None
 def _differential(c: VeroraxConfig, i: int, shapes) -> tuple[PartSpec, PartSpec | None]:
     m, where, prefix = c.layers[i].mixer, f"layers[{i}].mixer", f"l{i}.mix."
     return PartSpec("differential_attention", {
-        "hidden_size": c.width, **_heads(m, where), "dim": pos_int(m, "dim", where), "value_dim": pos_int(m, "vdim", where),
+        "hidden_size": c.width, **head_counts(m, where), "dim": pos_int(m, "dim", where), "value_dim": pos_int(m, "vdim", where),
         "scale": number(m, "scale", where), "diff": number(m, "diff", where), "eps": c.eps, "window": _window(m, where), "biases": True},
         prefix=prefix), None
 
@@ -145,7 +125,7 @@ def _side_by_side(c: VeroraxConfig, i: int, shapes) -> tuple[PartSpec, PartSpec 
     m, where, prefix = c.layers[i].mixer, f"layers[{i}].mixer", f"l{i}.mix."
     left, right = need(m, "left", where), need(m, "right", where)
     dim = pos_int(left, "dim", where + ".left")
-    lp = {"hidden_size": c.width, **_heads(left, where + ".left"), "key_dim": dim, "value_dim": pos_int(left, "vdim", where + ".left"),
+    lp = {"hidden_size": c.width, **head_counts(left, where + ".left"), "key_dim": dim, "value_dim": pos_int(left, "vdim", where + ".left"),
           "scale": number(left, "scale", where + ".left"), "eps": c.eps, "qk_norm": "weighted", "head_temperature": True,
           "window": _window(left, where + ".left"), "output_gate": "head"}
     position = _rotation(left, where + ".left", dim)

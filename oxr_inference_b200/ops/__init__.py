@@ -15,7 +15,7 @@ from __future__ import annotations
 import ctypes
 import functools
 import os
-from ctypes import c_float, c_int, c_longlong, c_size_t, c_void_p
+from ctypes import c_double, c_float, c_int, c_longlong, c_size_t, c_void_p
 
 import torch
 
@@ -113,7 +113,7 @@ def _lib():
         lib.oxr_gemm_f32_nt.argtypes = [p, p, p, i, i, i, p]
         lib.oxr_gemm_skinny_bf16.argtypes = [p, p, p, i, i, i, i, p]
         lib.oxr_gemm_skinny_gated_bf16.argtypes = [p, p, p, i, i, i, p]
-        lib.oxr_gemm_stream_bf16.argtypes = [p, p, p, i, i, i, i, p, p]
+        lib.oxr_gemm_stream_bf16.argtypes = [p, p, p, i, i, i, i, i, p, p]
         lib.oxr_gemm_stream_gated_bf16.argtypes = [p, p, p, i, i, i, p, p]
         lib.oxr_gemm_stream_add_bf16.argtypes = [p, p, p, p, p, p, p, i, i, i, p, p]
         lib.oxr_gemm_stream_add_bf16.restype = c_int
@@ -121,8 +121,8 @@ def _lib():
         lib.oxr_gemm_stream_scaled_bf16.restype = c_int
         lib.oxr_gemm_stream_blocks.argtypes = [i]
         lib.oxr_gemm_stream_blocks.restype = c_int
-        lib.oxr_gemm_tcgen05_bf16.argtypes = [p, p, p, i, i, i, i, i, i, p, p, p, p]
-        lib.oxr_gemm_tcgen05_pair_bf16.argtypes = [p, p, p, i, i, i, i, i, p, p]
+        lib.oxr_gemm_tcgen05_bf16.argtypes = [p, p, p, i, i, i, i, i, i, p, p, i, p, p]
+        lib.oxr_gemm_tcgen05_pair_bf16.argtypes = [p, p, p, i, i, i, i, i, i, p, p]
         lib.oxr_gemm_tcgen05_gated_bf16.argtypes = [p, p, p, i, i, i, i, p, p]
         lib.oxr_gemm_few_rows_cluster_bf16.argtypes = [p, p, p, i, i, i, i, i, p, p]
         lib.oxr_gemm_few_rows_max_clusters.argtypes = [i]
@@ -138,7 +138,7 @@ def _lib():
         lib.oxr_concat2_cast.argtypes = [p, p, p, i, i, i, p]
         lib.oxr_add_row_f32.argtypes = [p, p, i, i, p]
         lib.oxr_clamped_glu.argtypes = [p, p, i, i, i, f, f, i, p]
-        lib.oxr_rotary_angles.argtypes = [p, p, p, p, i, i, p]
+        lib.oxr_rotary_angles.argtypes = [p, p, p, p, c_double, i, i, p]
         lib.oxr_mamba_conv.argtypes = [p, p, i, i, i, i, i, i, p, p, p, ll, p, p, p, i, p]
         lib.oxr_mamba_scan.argtypes = [p, p, p, i, i, i, i, i, i, i, p, p, p, p, ll, p, p, i, p]
         lib.oxr_gated_group_norm.argtypes = [p, p, p, i, i, i, p, i, i, f, i, p]
@@ -152,7 +152,7 @@ def _lib():
         lib.oxr_scale_f32.argtypes = [p, f, ll, p]
         lib.oxr_mlstm_scan.argtypes = [p, p, p, i, i, i, i, i, p, p, i, i, i, f, f, p, ll, p, p, i, p]
         lib.oxr_head_norm_gate.argtypes = [p, p, p, i, i, i, p, i, i, f, i, i, p]
-        lib.oxr_route.argtypes = [p, p, p, p, i, i, i, i, i, f, i, i, i, p, i, p, p]
+        lib.oxr_route.argtypes = [p, p, p, p, i, i, i, i, i, f, i, i, i, p, i, p, p, p]
         lib.oxr_gated_relu2.argtypes = [p, p, p, i, i, i, i, p]
         lib.oxr_expert_sort.argtypes = [p, p, p, p, p, i, i, i, i, p]
         lib.oxr_gemm_tcgen05_grouped_bf16.argtypes = [p, p, p, i, i, i, i, p, i, i, i, p, p]
@@ -186,6 +186,8 @@ def _lib():
         lib.oxr_tanh_cols.argtypes = [p, p, i, i, i, i, i, p]
         lib.oxr_diff_prep.argtypes = [p, p, p, p, i, i, i, i, i, i, i, i, i, i, i, p, p, ll, i, p, p]
         lib.oxr_diff_combine.argtypes = [p, p, i, i, i, i, p, f, f, i, p]
+        lib.oxr_hyper_mix.argtypes = [p, p, p, ll, ll, p, p, p, p, p, p, p, f, i, i, i, i, p]
+        lib.oxr_hyper_mix.restype = c_int
         for name in ("oxr_head_prep", "oxr_sigmoid_gate", "oxr_gla_scan", "oxr_pair_norm_mean", "oxr_tanh_cap", "oxr_expert_silu_glu",
                      "oxr_scale_placed_rows", "oxr_add_row_gated", "oxr_cols_rms_norm", "oxr_gelu_glu", "oxr_scaled_sum", "oxr_shift_norm",
                      "oxr_delta_scan", "oxr_tanh_cols", "oxr_diff_prep", "oxr_diff_combine"):
@@ -611,7 +613,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         raise KernelError(f"no tile list for long tiles of {long_rows} rows: the batch was cut for {sorted(tiles)}")
     s_req, s_tok, n_short = tiles[short]
     l_req, l_tok, n_long = tiles[long_]
-    splits, cut, part_o, part_ml, counters = _split_kv_plan(lib, n_short, num_heads, num_kv_heads, head_dim, kv_len_bound, kv_maps is not None,
+    seen = kv_len_bound if window <= 0 else min(kv_len_bound, window + keep_first + SHORT_MAX_TOKENS)     # keys a short tile can see
+    splits, cut, part_o, part_ml, counters = _split_kv_plan(lib, n_short, num_heads, num_kv_heads, head_dim, seen, kv_maps is not None,
                                                             uneven, q.device)
     if masked:
         for t, nm in ((dist_bias, "dist_bias"), (sink, "sink")):
@@ -924,7 +927,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None 
         raise KernelError(f"linear: activations {x.dtype} with weight {weight.dtype} is not a supported pair")
     if STREAM_GEMM and m <= STREAM_MAX_ROWS and k % 8 == 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0:
         out = given if given is not None else torch.empty((m, n), dtype=out_dtype, device=x.device)
-        _done(lib.oxr_gemm_stream_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, _DT[out_dtype],
+        _done(lib.oxr_gemm_stream_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, _DT[out_dtype], 0,
                                        new_status(x.device).data_ptr(), _stream()), "gemm_stream")
         return out
     if m <= SKINNY_MAX_ROWS and k % 8 == 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0:
@@ -941,7 +944,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None 
             return out
         pair_tile = _gemm_pair_plan(m, n, k)
         if pair_tile:
-            _done(lib.oxr_gemm_tcgen05_pair_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, _DT[out_dtype], pair_tile,
+            _done(lib.oxr_gemm_tcgen05_pair_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, _DT[out_dtype], pair_tile, 0,
                                                  new_status(x.device).data_ptr(), _stream()), "gemm_tcgen05_pair")
             return out
         tile_n, splits = _gemm_plan(m, n, k)
@@ -951,7 +954,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None 
                 raise KernelError(f"linear: {splits} shares of {m} x {n} in tiles of {tile_n} columns outgrow the workspace")
             partial, tickets = _gemm_split_buffers(x.device)
         code = lib.oxr_gemm_tcgen05_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, _DT[out_dtype], tile_n, splits,
-                                         _ptr(partial), _ptr(tickets), new_status(x.device).data_ptr(), _stream())
+                                         _ptr(partial), _ptr(tickets), 0, new_status(x.device).data_ptr(), _stream())
         _done(code, "gemm_tcgen05")
         return out
     # rows that are not whole 16-byte words cannot be fetched by TMA: the library product takes them
@@ -960,6 +963,39 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None 
         given.copy_(got)
         return given
     return got
+
+
+def relu2_linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``relu(x @ weight.T)^2`` in x's dtype. bfloat16: the epilogue of the kernel that ``linear`` would pick applies the activation to the fp32 sums for
+    decode-sized products and from ``GEMM_PAIR_MIN_ROWS`` rows on, and wherever the one-SM kernel takes the product whole; the sizes in between,
+    where k is dealt out in shares, and float32 run the product and then the activation kernel."""
+    _need(x, "x")
+    _need(weight, "weight")
+    m, k = x.shape
+    n = weight.shape[0]
+    if weight.shape[1] != k:
+        raise KernelError(f"relu2_linear: x has {k} columns, weight has {weight.shape[1]}")
+    if x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and k % 8 == 0 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0:
+        lib, status = _lib(), new_status(x.device).data_ptr()
+        pair_tile = _gemm_pair_plan(m, n, k)
+        if m <= STREAM_MAX_ROWS and STREAM_GEMM:
+            out = torch.empty((m, n), dtype=x.dtype, device=x.device)
+            _done(lib.oxr_gemm_stream_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, 1, 1, status, _stream()), "gemm_stream")
+            return out
+        if pair_tile:
+            out = torch.empty((m, n), dtype=x.dtype, device=x.device)
+            _done(lib.oxr_gemm_tcgen05_pair_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, 1, pair_tile, 1, status, _stream()),
+                  "gemm_tcgen05_pair")
+            return out
+        if m > SKINNY_MAX_ROWS and not _gemm_few_rows_plan(m, n, k):
+            tile_n, splits = _gemm_plan(m, n, k)
+            if splits == 1:
+                out = torch.empty((m, n), dtype=x.dtype, device=x.device)
+                _done(lib.oxr_gemm_tcgen05_bf16(out.data_ptr(), x.data_ptr(), weight.data_ptr(), m, n, k, 1, tile_n, 1, None, None, 1, status, _stream()),
+                      "gemm_tcgen05")
+                return out
+    u = linear(x, weight)
+    return gated_relu2(u, None, n, out=u)
 
 
 FUSE_MAX_ROWS = min(16, int(os.environ.get("OXR_B200_FUSE_ROWS", "16")))
@@ -1158,15 +1194,15 @@ def gelu_glu(gate_up: torch.Tensor, interleave: int = 0) -> torch.Tensor:
     return out
 
 
-def rotary_angles(positions: torch.Tensor, freq: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    """fp32 ``cos`` and ``sin`` ``[tokens, len(freq)]`` of ``position * freq[i]`` for this step's tokens; the product and the functions are
-    evaluated in fp64 (``freq`` is a float64 device tensor) and rounded once, so the table is exact to fp32 at any position."""
+def rotary_angles(positions: torch.Tensor, freq: torch.Tensor, magnitude: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """fp32 ``cos`` and ``sin`` ``[tokens, len(freq)]`` of ``position * freq[i]``, times ``magnitude``, for this step's tokens; products and functions
+    are evaluated in fp64 (``freq`` is a float64 device tensor) and rounded once, so the table is exact to fp32 at any position."""
     _need(positions, "positions", torch.int32)
     _need(freq, "freq", torch.float64)
     n, half = positions.numel(), freq.numel()
     cos = torch.empty((n, half), dtype=torch.float32, device=positions.device)
     sin = torch.empty_like(cos)
-    _done(_lib().oxr_rotary_angles(cos.data_ptr(), sin.data_ptr(), positions.data_ptr(), freq.data_ptr(), n, half, _stream()), "rotary_angles")
+    _done(_lib().oxr_rotary_angles(cos.data_ptr(), sin.data_ptr(), positions.data_ptr(), freq.data_ptr(), float(magnitude), n, half, _stream()), "rotary_angles")
     return cos, sin
 
 
@@ -1675,15 +1711,16 @@ def head_norm_gate(y: torch.Tensor, proj: torch.Tensor, gate_col0: int, weight: 
 
 
 # --------------------------------------------------------------------------------------------------- routed experts
-ROUTE_SCORES = {"sigmoid": 0, "softmax": 1}
+ROUTE_SCORES = {"sigmoid": 0, "softmax": 1, "chosen_softmax": 2}
 ROUTE_GROUP_SCORES = {"top2_sum": 0, "max": 1}
 
 
 def route(z: torch.Tensor, *, top: int, groups: int, keep: int, scale: float, score: str = "sigmoid", group_score: str = "top2_sum",
           renormalize: bool = True, correction: torch.Tensor | None = None,
-          kept: torch.Tensor | None = None, identity: int = 0) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
-    """Router logits ``z [tokens, E]`` (fp32) to the choice of ``top`` experts per token. Scores are ``sigmoid(z)`` or, with ``score="softmax"``,
-    the softmax of z over all experts; of ``groups`` equal groups of neighbouring experts only the ``keep`` best may be chosen from, a group's
+          kept: torch.Tensor | None = None, identity: int = 0, bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """Router logits ``z [tokens, E]`` (fp32; plus ``bias [E]``, fp32, where given) to the choice of ``top`` experts per token. Scores are ``sigmoid(z)`` or,
+    with ``score="softmax"``, the softmax of z over all experts; with ``"chosen_softmax"`` groups and experts are picked by the logits themselves and
+    the weights are the softmax over the chosen logits (``renormalize`` is then a must). Of ``groups`` equal groups of neighbouring experts only the ``keep`` best may be chosen from, a group's
     score being the sum of its two best scores (``"top2_sum"``) or its best score (``"max"``); the weights are the chosen scores over their sum
     (``renormalize``) or as they are, times ``scale``. With ``correction [E]`` (fp32) groups and experts are chosen by score + correction; the weights
     stay those of the scores. The last ``identity`` of the E experts return their input: the sum of a token's weights for them goes to ``kept
@@ -1697,6 +1734,12 @@ def route(z: torch.Tensor, *, top: int, groups: int, keep: int, scale: float, sc
         _need(correction, "correction", torch.float32)
         if correction.numel() != E:
             raise KernelError("route: one correction per expert")
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        if bias.numel() != E:
+            raise KernelError("route: one bias per expert")
+    if score == "chosen_softmax" and (not renormalize or correction is not None):
+        raise KernelError("route: the softmax over the chosen logits is normalised and takes no correction")
     gate = torch.empty((n, E - identity), dtype=torch.float32, device=z.device)
     if identity:
         _need(kept, "kept", torch.float32)
@@ -1706,7 +1749,7 @@ def route(z: torch.Tensor, *, top: int, groups: int, keep: int, scale: float, sc
     wts = torch.empty((n, top), dtype=torch.float32, device=z.device)
     _done(_lib().oxr_route(gate.data_ptr(), ids.data_ptr(), wts.data_ptr(), z.data_ptr(), n, E, int(top), int(groups), int(keep), float(scale),
                            ROUTE_SCORES[score], ROUTE_GROUP_SCORES[group_score], int(bool(renormalize)), _ptr(correction), E - identity,
-                           _ptr(kept) if identity else None, _stream()), "route")
+                           _ptr(kept) if identity else None, _ptr(bias), _stream()), "route")
     return gate, ids, wts
 
 
@@ -2044,6 +2087,58 @@ def shift_norm(stream: torch.Tensor, weight: torch.Tensor, eps: float, shift: to
                                 weight.data_ptr(), float(eps), shift.data_ptr(), state.data_ptr(), state.stride(0), req_of_token.data_ptr(), cu_q.data_ptr(),
                                 state_slots.data_ptr(), n, hidden, int(rows), _DT[out_dtype], _stream()), "shift_norm")
     return out, new
+
+
+# --------------------------------------------------------------------------------------------------- several residual streams
+HYPER_MAX_STREAMS = 16
+
+
+def hyper_mix(x: torch.Tensor, streams: int, out_dtype: torch.dtype, *, y: torch.Tensor | None = None, mix: torch.Tensor | None = None,
+              out_weights: torch.Tensor | None = None, scale: torch.Tensor | None = None,
+              then: tuple[torch.Tensor, torch.Tensor, float] | None = None) -> tuple[torch.Tensor | None, torch.Tensor]:
+    """What stands between two sublayers of ``streams`` residual streams, in one kernel. ``x``: the streams, fp32 ``[tokens, streams, hidden]``, or ``[tokens,
+    hidden]`` when all are equal (in front of the first sublayer). With a sublayer's result ``y [tokens, hidden]`` (``out_dtype``) the streams become
+
+        x_t <- sum_s mix[s, t] x_s + out_weights[t] * (scale * y)          (``scale [hidden]`` is optional)
+
+    in place, or in a new tensor when x holds one copy. ``then = (in_weights [streams], norm weight [hidden], eps)``: also returns the next sublayer's
+    input ``h = u / rms(u) * weight`` with ``u = sum_t in_weights[t] x_t`` in ``out_dtype``: ``(h, streams)``. Without ``then`` the streams end here:
+    ``(None, sum_t x_t)`` as ``[tokens, hidden]``, and x stays as it was."""
+    _need(x, "x", torch.float32)
+    n, hidden, S = x.shape[0], x.shape[-1], int(streams)
+    whole = x.dim() == 3
+    if (whole and x.shape[1] != S) or x.dim() not in (2, 3) or not 1 <= S <= HYPER_MAX_STREAMS:
+        raise KernelError(f"hyper_mix: {tuple(x.shape)} is not {S} streams")
+    if y is None and then is None:
+        raise KernelError("hyper_mix: nothing to do")
+    if y is not None:
+        _need(y, "y", out_dtype)
+        _need(mix, "mix", torch.float32)
+        _need(out_weights, "out_weights", torch.float32)
+        if y.shape != (n, hidden) or mix.shape != (S, S) or out_weights.numel() != S:
+            raise KernelError("hyper_mix: the sublayer's result or its weights do not fit the streams")
+        if scale is not None:
+            _need(scale, "scale", torch.float32)
+            if scale.numel() != hidden:
+                raise KernelError("hyper_mix: one scale per entry")
+    h = in_w = weight = total = None
+    eps = 0.0
+    new = x
+    if then is not None:
+        in_w, weight, eps = then
+        _need(in_w, "in_weights", torch.float32)
+        _need(weight, "norm weight", torch.float32)
+        if in_w.numel() != S or weight.numel() != hidden:
+            raise KernelError("hyper_mix: one weight per stream, one norm weight per entry")
+        h = torch.empty((n, hidden), dtype=out_dtype, device=x.device)
+        if y is not None and not whole:
+            new = torch.empty((n, S, hidden), dtype=torch.float32, device=x.device)
+    else:
+        total = torch.empty((n, hidden), dtype=torch.float32, device=x.device)
+    _done(_lib().oxr_hyper_mix(_ptr(h), _ptr(y), x.data_ptr(), S * hidden if whole else hidden, hidden if whole else 0,
+                               new.data_ptr() if y is not None and then is not None else None, _ptr(total), _ptr(mix), _ptr(out_weights), _ptr(scale),
+                               _ptr(in_w), _ptr(weight), float(eps), n, S, hidden, _DT[out_dtype], _stream()), "hyper_mix")
+    return h, (new if then is not None else total)
 
 
 # --------------------------------------------------------------------------------------------------- delta rule

@@ -191,6 +191,98 @@ class PendingNormedAdd:
         self.y, self.norm = y, norm
 
 
+@ARRANGEMENTS.register("hyper_connections")
+class HyperConnectedBlock(Part):
+    """Pre-norm sublayers on ``streams`` residual streams x_1 .. x_s beside each other (hyper-connections). A sublayer q (1: the mixer, 2: the
+    feed-forward, when the block has one) reads ``u = sum_s in[s] x_s`` through its norm, and its result y changes all streams at once:
+
+        x_t <- sum_s mix[s, t] x_s + out[t] * (scale * y)
+
+    with tensors ``hc<q>.in [streams]``, ``hc<q>.out [streams]``, ``hc<q>.mix [streams, streams]`` and, with ``layer_scale``, ``ls<q> [hidden]`` (without:
+    scale = 1). The first block of a run of such blocks takes the one stream it is handed as all of them; the last one hands on their sum.
+
+    In between, ``forward`` passes the fp32 streams ``[tokens, streams, hidden]`` in ``residual`` and leaves its last result to the next block
+    (:class:`PendingStreamUpdate`): the update of the streams and the norm that reads them next are one kernel, so a block costs two launches beside its
+    sublayers."""
+
+    def __init__(self, mixer: Mixer, mixer_norm: Norm, feed_forward: FeedForward | None, feed_forward_norm: Norm | None, *, runtime: Runtime,
+                 hidden_size: int, streams: int, layer_scale: bool = False):
+        if (feed_forward is None) != (feed_forward_norm is None):
+            raise ValueError("a feed-forward comes with its norm or not at all")
+        for norm in (mixer_norm, feed_forward_norm):
+            if norm is not None and not hasattr(norm, "of_streams"):
+                raise ValueError("the hyper_connections arrangement is built for norms that offer of_streams (rms_norm)")
+        if not 1 <= int(streams) <= ops.HYPER_MAX_STREAMS:
+            raise ValueError(f"{streams} streams: 1 to {ops.HYPER_MAX_STREAMS} are built")
+        self.runtime, self.hidden, self.streams, self.layer_scale = runtime, int(hidden_size), int(streams), bool(layer_scale)
+        self.mixer, self.mixer_norm, self.feed_forward, self.feed_forward_norm = mixer, mixer_norm, feed_forward, feed_forward_norm
+        self.vectors: dict[str, torch.Tensor] = {}
+
+    def parts(self) -> dict[str, object]:
+        out = {"mixer": self.mixer, "mixer_norm": self.mixer_norm}
+        if self.feed_forward is not None:
+            out.update(feed_forward=self.feed_forward, feed_forward_norm=self.feed_forward_norm)
+        return out
+
+    def parameters(self) -> dict[str, ParamInfo]:
+        s = self.streams
+        out: dict[str, ParamInfo] = {}
+        for q in (1, 2) if self.feed_forward is not None else (1,):
+            for name, shape in (("in", (s,)), ("out", (s,)), ("mix", (s, s))):
+                out[f"hc{q}.{name}"] = ParamInfo(shape, role="vector")
+            if self.layer_scale:
+                out[f"ls{q}"] = ParamInfo((self.hidden,), role="vector")
+        return out
+
+    def assign(self, name: str, tensor: torch.Tensor) -> None:
+        if name not in self.parameters():
+            raise KeyError(name)
+        self.vectors[name] = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
+
+    def keeps_add_for(self, after) -> bool:
+        """Whether ``after`` (the block that runs next, or None) goes on with the same streams and takes this block's last update into its first norm."""
+        return isinstance(after, HyperConnectedBlock) and after.streams == self.streams
+
+    def _update(self, q: int, y: torch.Tensor) -> "PendingStreamUpdate":
+        v = self.vectors
+        return PendingStreamUpdate(self, ops.cast(y, self.runtime.dtype), v[f"hc{q}.mix"], v[f"hc{q}.out"], v.get(f"ls{q}"))
+
+    def forward(self, x, residual: torch.Tensor | None, ctx: StepContext, cache: LayerCache, defer_output: bool = False):
+        pending = None
+        if isinstance(x, PendingStreamUpdate):
+            pending, streams = x, residual
+        elif residual is None:
+            if isinstance(x, DeferredLinear):
+                x = x.materialize()
+            if x.dtype != torch.float32:
+                raise ValueError("this arrangement keeps the streams in fp32: the embedding must hand its output over whole")
+            streams = x
+        elif x is not None:
+            raise ValueError("this arrangement takes the stream whole; the block before it left an output that is not yet added")
+        else:
+            streams = residual
+        h, streams = self.mixer_norm.of_streams(streams, self.streams, self.vectors["hc1.in"], pending.args if pending is not None else None)
+        last = self._update(1, self.mixer.forward(h, ctx, cache))
+        if self.feed_forward is not None:
+            h, streams = self.feed_forward_norm.of_streams(streams, self.streams, self.vectors["hc2.in"], last.args)
+            last = self._update(2, self.feed_forward.forward(h))
+        if defer_output:
+            return last, streams
+        return None, last.total(streams)
+
+
+class PendingStreamUpdate:
+    """A sublayer's result that has not yet reached the streams of a :class:`HyperConnectedBlock`."""
+
+    def __init__(self, block: HyperConnectedBlock, y: torch.Tensor, mix: torch.Tensor, out_weights: torch.Tensor, scale: torch.Tensor | None):
+        self.block = block
+        self.args = dict(y=y, mix=mix, out_weights=out_weights, scale=scale)
+
+    def total(self, streams: torch.Tensor) -> torch.Tensor:
+        """The sum of the streams as they are after the update (``streams`` stays as it is): what a run of such blocks hands on."""
+        return ops.hyper_mix(streams, self.block.streams, self.block.runtime.dtype, **self.args)[1]
+
+
 @ARRANGEMENTS.register("output_norm")
 class OutputNormBlock:
     """``x += norm1(mixer(x))`` and, when the block has a feed-forward, ``x += norm2(ff(x))``: the sublayers read the stream itself and the only

@@ -17,7 +17,8 @@ class RoutedExperts(FeedForward):
     ``u = clamp(up_i h, -limit, limit)`` (``"clamped_glu"``) or the SiLU-gated unit ``down_i( silu(gate_i h) * (up_i h) )`` (``"silu_glu"``). The router's logits ``z = W_router h`` are computed in fp32; scores
     ``s = sigmoid(z)`` or the softmax of z over all experts (``score``). The experts form ``groups`` equal groups of neighbours; a group's
     score is the sum of its two largest scores or its largest one (``group_score``), and only experts of the ``keep`` best groups can be
-    chosen. Each token runs the ``top`` allowed experts with the largest scores; their outputs are added with weights
+    chosen. ``score="chosen_softmax"``: groups and experts are picked by the logits, the weights are the softmax over the chosen logits alone.
+    ``router_bias``: a learned number per expert (tensor ``router.b``) joins the logits. Each token runs the ``top`` allowed experts with the largest scores; their outputs are added with weights
     ``s / (sum of the chosen s + 1e-20) * scale`` or, with ``renormalize=False``, ``s * scale``. ``choice_correction``: a learned number per expert
     (tensor ``correction``) is added to the scores for the choice (of groups and experts) and nowhere else. ``identity``: that many more experts
     behind the others are scored and chosen like them but have no tensors and return their input. With ``weight_on="input"`` the weight multiplies
@@ -41,7 +42,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, runtime: Runtime, *, hidden_size: int, intermediate_size: int, experts: int, top: int, groups: int = 1, keep: int = 1,
                  scale: float = 1.0, grouped_min_rows: int | None = None, activation: str = "relu2", limit: float = 0.0, alpha: float = 1.702,
                  score: str = "sigmoid", group_score: str = "top2_sum", renormalize: bool = True, shared: Mapping[str, Any] | None = None,
-                 weight_on: str = "output", shared_gate: bool = False, choice_correction: bool = False, identity: int = 0):
+                 weight_on: str = "output", shared_gate: bool = False, choice_correction: bool = False, identity: int = 0,
+                 router_bias: bool = False):
         self.runtime = runtime
         if activation not in ("relu2", "clamped_glu", "silu_glu"):
             raise ValueError(f"expert activation {activation!r} is not one of 'relu2', 'clamped_glu', 'silu_glu'")
@@ -65,6 +67,9 @@ class RoutedExperts(FeedForward):
         self.groups, self.keep, self.scale = int(groups), int(keep), float(scale)
         self.identity, self.scored = int(identity), int(experts) + int(identity)
         self.has_correction, self.correction = bool(choice_correction), None
+        self.has_bias, self.router_bias = bool(router_bias), None
+        if self.score == "chosen_softmax" and (self.has_correction or not self.renormalize):
+            raise ValueError("the softmax over the chosen logits is normalised and takes no correction")
         if self.groups < 1 or self.scored % self.groups:
             raise ValueError(f"{self.scored} experts do not form {self.groups} equal groups")
         if not 1 <= self.keep <= self.groups:
@@ -82,6 +87,8 @@ class RoutedExperts(FeedForward):
         out = {"router": ParamInfo((self.scored, self.hidden))}
         if self.has_correction:
             out["correction"] = ParamInfo((self.scored,), role="vector")
+        if self.has_bias:
+            out["router.b"] = ParamInfo((self.scored,), role="vector")
         for e in range(self.E):
             if self.gated:
                 out[f"e{e}.gate"] = ParamInfo((self.ff, self.hidden))
@@ -116,6 +123,9 @@ class RoutedExperts(FeedForward):
         if name == "correction" and self.has_correction:
             self.correction = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
             return
+        if name == "router.b":
+            self.router_bias = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
+            return
         expert, which = name.split(".")
         e = int(expert[1:])
         if which in ("up", "gate"):
@@ -143,7 +153,7 @@ class RoutedExperts(FeedForward):
         kept = torch.empty((h.shape[0],), dtype=torch.float32, device=h.device) if self.identity else None
         gate, ids, weights = ops.route(z, top=self.top, groups=self.groups, keep=self.keep, scale=self.scale, score=self.score,
                                        group_score=self.group_score, renormalize=self.renormalize, correction=self.correction, kept=kept,
-                                       identity=self.identity)
+                                       identity=self.identity, bias=self.router_bias)
         if self.top < self.scored and h.shape[0] >= self.grouped_min_rows > 0 and not torch.cuda.is_current_stream_capturing():
             y = self._grouped(h, ids, weights, kept)
         else:

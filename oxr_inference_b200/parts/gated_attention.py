@@ -48,6 +48,8 @@ class GatedAttention(Mixer):
             raise ValueError(f"output_gate {output_gate!r} is not one of None, 'channel', 'head'")
         if position is not None and not hasattr(position, "step_angles"):
             raise ValueError("gated_attention rotates by per-step angles (a position encoding with step_angles)")
+        if position is not None and not getattr(position, "halves", True):
+            raise ValueError("gated_attention turns the pairs (i, i + half), not neighbours")
         if position is not None and position.dims > key_dim:
             raise ValueError(f"{position.dims} rotated entries do not fit heads of {key_dim}")
         if values_are_keys and value_dim != key_dim:

@@ -224,7 +224,8 @@ class LatentAttention(Mixer):
     the latent ``c`` and ``rot_dim`` more that are rotated into a key part shared by all heads; only ``[c | rotated part]`` is
     cached. Per head the unrotated key is ``W_uk c`` and the value ``W_uv c``; the query ``W_q h`` is laid out head by head as
     ``[key_dim unrotated | rot_dim rotated]``; the score is ``(q_u . k_u + q_r . k_r) * scale``; causal; optional ``sink``: a learned
-    number per head whose exponential joins the softmax denominator (it has no key, no value and is not scaled). ``q_rank`` > 0: the query
+    number per head whose exponential joins the softmax denominator (it has no key, no value and is not scaled). ``window`` > 0: position i sees
+    only its last ``window`` positions, itself among them (pages behind that are given back). ``q_rank`` > 0: the query
     passes a latent of its own, ``W_uq rmsnorm(W_dq h)`` with the weight ``dq.norm`` (tensors ``dq``, ``dq.norm``, ``uq`` in place of ``q``). Which entries
     of the rotated part form a pair is the position encoding's (neighbours, or an entry and the one half the rotated part further on).
 
@@ -233,12 +234,12 @@ class LatentAttention(Mixer):
     well), and ``W_uv`` is applied to the attention's output."""
 
     def __init__(self, runtime: Runtime, position: PositionEncoding | None, *, hidden_size: int, num_heads: int, key_dim: int, rot_dim: int,
-                 value_dim: int, rank: int, scale: float, eps: float, sink: bool = True, q_rank: int = 0):
+                 value_dim: int, rank: int, scale: float, eps: float, sink: bool = True, q_rank: int = 0, window: int = 0):
         if rot_dim and position is None:
             raise ValueError("latent_attention with a rotated part needs a position encoding")
         self.runtime, self.position = runtime, position
         self.hidden, self.H, self.D, self.R, self.DV, self.L = int(hidden_size), int(num_heads), int(key_dim), int(rot_dim), int(value_dim), int(rank)
-        self.scale, self.eps, self.has_sink = float(scale), float(eps), bool(sink)
+        self.scale, self.eps, self.has_sink, self.window = float(scale), float(eps), bool(sink), int(window)
         self.QL, q_cols = int(q_rank), self.H * (self.D + self.R)
         # everything that reads h is one product
         self.q_dkv = StackedLinear(runtime, self.hidden, {**({"dq": self.QL} if self.QL else {"q": q_cols}), "dkv": self.L + self.R})
@@ -285,7 +286,7 @@ class LatentAttention(Mixer):
             raise KeyError(name)
 
     def cache_need(self) -> PagedKVNeed:
-        return PagedKVNeed(1, self.L + self.R, 0, value_dim=0)
+        return PagedKVNeed(1, self.L + self.R, self.window, value_dim=0)
 
     @property
     def tiled(self) -> bool:
@@ -323,12 +324,12 @@ class LatentAttention(Mixer):
         ops.head_linear(q_abs, 0, q, 0, self.uk)
         if self.tiled and pool.dtype == torch.bfloat16:
             o_lat = ops.paged_attention(q_abs, pool, pool, tiles=ctx.tiles, cu_q=ctx.cu_q, ctx_lens=ctx.ctx_lens, block_table=group.block_table,
-                                        page_size=group.page_size, scale=self.scale, window=0, kv_len_bound=ctx.kv_len_bound, status=ctx.status,
-                                        sink=self.sink)                       # [n, H, L + R]: the first L entries are the latent output
+                                        page_size=group.page_size, scale=self.scale, window=self.window, kv_len_bound=ctx.kv_len_bound,
+                                        status=ctx.status, sink=self.sink)                       # [n, H, L + R]: the first L entries are the latent output
         else:
             o_lat = ops.attention_rows(q_abs.view(n, H * (L + R)), H, pool, None, value_dim=L, positions=ctx.positions,
-                                       req_of_token=ctx.req_of_token, block_table=group.block_table, scale=self.scale, sink=self.sink,
-                                       status=ctx.status).view(n, H, L)
+                                       req_of_token=ctx.req_of_token, block_table=group.block_table, scale=self.scale, window=self.window,
+                                       sink=self.sink, status=ctx.status).view(n, H, L)
         o = torch.empty((n, H, self.DV), dtype=pool.dtype, device=pool.device)
         ops.head_linear(o, 0, o_lat, 0, self.uv)
         return self.out(o.view(n, H * self.DV))

@@ -1,4 +1,4 @@
-"""Dense feed-forwards: SiLU-gated, clamped gated, GELU-gated, and a plain two-matrix layer with the tanh form of GELU."""
+"""Dense feed-forwards: SiLU-gated, clamped gated, GELU-gated, and plain two-matrix layers with the tanh form of GELU or the square of relu."""
 
 from __future__ import annotations
 
@@ -98,10 +98,8 @@ class GeluGLU(FeedForward):
         return self.down(ops.gated_linear(h, self.gate_up.weight, self.gate_up.interleave, kind="gelu"))
 
 
-@FEED_FORWARDS.register("gelu_mlp")
-class GeluMLP(FeedForward):
-    """``down( gelu_tanh(h W_up^T) )`` with ``gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``: two matrices, no gate, no
-    biases. The activation is evaluated in fp32 on the product's rounded output."""
+class TwoMatrixMLP(FeedForward):
+    """``down( act(h W_up^T) )``: two matrices, no gate, no biases."""
 
     def __init__(self, runtime: Runtime, *, hidden_size: int, intermediate_size: int):
         self.hidden, self.inter = int(hidden_size), int(intermediate_size)
@@ -120,4 +118,23 @@ class GeluMLP(FeedForward):
             raise KeyError(name)
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        return self.down(ops.gelu_tanh_(self.up(h)))
+        return self.down(self._hidden(h))
+
+    def _hidden(self, h: torch.Tensor) -> torch.Tensor:
+        raise NotImplementedError
+
+
+@FEED_FORWARDS.register("gelu_mlp")
+class GeluMLP(TwoMatrixMLP):
+    """``act = gelu_tanh``: ``0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``, evaluated in fp32 on the product's rounded output."""
+
+    def _hidden(self, h: torch.Tensor) -> torch.Tensor:
+        return ops.gelu_tanh_(self.up(h))
+
+
+@FEED_FORWARDS.register("relu2_mlp")
+class SquaredReluMLP(TwoMatrixMLP):
+    """``act = relu(z)^2``, in the product's epilogue where the kernel that takes the size has one."""
+
+    def _hidden(self, h: torch.Tensor) -> torch.Tensor:
+        return ops.relu2_linear(h, self.up.weight)

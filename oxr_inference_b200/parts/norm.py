@@ -11,19 +11,21 @@ from oxr_inference_b200.parts.base import NORMS, DeferredLinear, Norm, ParamInfo
 @NORMS.register("rms_norm")
 class RMSNorm(Norm):
     """``out = (x + residual) * rsqrt(mean((x + residual)^2) + eps) * weight`` with the sum kept as the new fp32
-    residual (oxr_runtime/language.py:69-72,94-99; layer 0 has no residual yet, language.py:253-257)."""
+    residual (oxr_runtime/language.py:69-72,94-99; layer 0 has no residual yet, language.py:253-257). ``around_zero``: the checkpoint stores
+    the weight's distance from one (the factor is ``1 + weight``, added in fp32 at load)."""
 
-    def __init__(self, runtime: Runtime, *, size: int, eps: float):
-        self.runtime, self.size, self.eps = runtime, int(size), float(eps)
+    def __init__(self, runtime: Runtime, *, size: int, eps: float, around_zero: bool = False):
+        self.runtime, self.size, self.eps, self.around_zero = runtime, int(size), float(eps), bool(around_zero)
         self.weight: torch.Tensor | None = None
 
     def parameters(self) -> dict[str, ParamInfo]:
-        return {"weight": ParamInfo((self.size,), init="around_one", role="vector")}
+        return {"weight": ParamInfo((self.size,), init="normal" if self.around_zero else "around_one", role="vector")}
 
     def assign(self, name: str, tensor: torch.Tensor) -> None:
         if name != "weight":
             raise KeyError(name)
-        self.weight = tensor.to(device=self.runtime.device, dtype=torch.float32).contiguous()
+        weight = tensor.to(device=self.runtime.device, dtype=torch.float32)
+        self.weight = (weight + 1.0 if self.around_zero else weight).contiguous()
 
     accepts_deferred = True
 
@@ -61,6 +63,10 @@ class RMSNorm(Norm):
             return ops.norm_add_norm(stream, y, self.weight, self.eps, rounded=rounded)
         return ops.norm_add_norm(stream, y, self.weight, self.eps, then.weight, then.eps)
 
+    def of_streams(self, streams: torch.Tensor, count: int, in_weights: torch.Tensor, pending: dict | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+        """``rmsnorm(sum_s in_weights[s] x_s) * weight`` of ``count`` residual streams in the activation dtype, and the streams; ``pending`` (``y``, ``mix``,
+        ``out_weights``, ``scale``: a sublayer's result that has not yet reached the streams) is added in the same pass."""
+        return ops.hyper_mix(streams, count, self.runtime.dtype, then=(in_weights, self.weight, self.eps), **(pending or {}))
 
     def shifted(self, stream: torch.Tensor, shift: torch.Tensor, state: torch.Tensor, ctx: StepContext, pending=None) -> tuple[torch.Tensor, torch.Tensor]:
         """``h = rmsnorm(stream) * weight`` blended with the token before, ``h + (h' - h) * shift``, in the activation dtype; ``state`` holds h' of each

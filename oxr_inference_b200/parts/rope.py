@@ -1,4 +1,4 @@
-"""Rotary position encodings: the half-split (GPT-NeoX) table, and per-step angles for the interleaved-pairs form."""
+"""Rotary position encodings: the half-split (GPT-NeoX) table, and per-step angles for interleaved and half-split pairs."""
 
 from __future__ import annotations
 
@@ -31,30 +31,6 @@ class RotaryTable(PositionEncoding):
 
     def tables(self) -> tuple[torch.Tensor, torch.Tensor]:
         return self.cos, self.sin
-
-
-@POSITION_ENCODINGS.register("rope_pairs")
-class RotaryPairs(PositionEncoding):
-    """Rotary encoding of entry pairs (2i, 2i+1) of the first ``dims`` entries of a vector: the pair (u, v) at position p becomes
-    ``(u cos a - v sin a, v cos a + u sin a)`` with ``a = p * base^(-2i/dims)``. There is no table over all positions: each step
-    computes cos and sin for its own tokens, once, shared by every layer with the same ``dims`` and ``base`` (the frequencies, the
-    product with the position and the functions in fp64, rounded once to fp32), so no position limit comes from here."""
-
-    def __init__(self, runtime: Runtime, *, dims: int, base: float):
-        if dims % 2 or dims <= 0:
-            raise ValueError(f"rotary dimension {dims} must be even and positive")
-        self.dims, self.base = int(dims), float(base)
-        freq = torch.tensor([self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)], dtype=torch.float64)
-        self.freq = freq.to(runtime.device)
-
-    def tables(self):
-        raise NotImplementedError("rope_pairs has per-step angles (step_angles), not a table over all positions")
-
-    def step_angles(self, ctx: StepContext) -> tuple[torch.Tensor, torch.Tensor]:
-        key = ("rope_pairs", self.dims, self.base)
-        if key not in ctx.shared:
-            ctx.shared[key] = ops.rotary_angles(ctx.positions, self.freq)
-        return ctx.shared[key]
 
 
 def banded_frequencies(freq: list[float], *, factor: float, low: float, high: float, original: float) -> list[float]:
@@ -90,17 +66,16 @@ def ramped_frequencies(freq: list[float], *, dims: int, base: float, factor: flo
     return out, 0.1 * math.log(factor) + 1.0
 
 
-@POSITION_ENCODINGS.register("rope_halves")
-class RotaryHalves(PositionEncoding):
-    """Rotary encoding of the first ``dims`` entries of a vector in the half-split layout: entry i is paired with entry ``i + dims / 2`` and the
-    pair (u, v) at position p becomes ``(u cos a - v sin a, v cos a + u sin a)`` with ``a = p * f_i``, ``f_i = base^(-2i/dims)``. ``scaling``
-    rescales the frequencies: ``{"kind": "bands", factor, low, high, original}`` (:func:`banded_frequencies`) or ``{"kind": "ramp", factor,
-    original, fast, slow}`` (:func:`ramped_frequencies`, which also multiplies cos and sin by a constant). Like ``rope_pairs`` it has no
-    table over positions: each step computes cos and sin ``[tokens, dims / 2]`` for its own tokens once (frequencies, product and functions in
-    fp64, rounded once to fp32) and layers with equal parameters share them."""
+class StepAngles(PositionEncoding):
+    """Rotary encoding of the first ``dims`` entries of a vector: pair i, (u, v), at position p becomes ``(u cos a - v sin a, v cos a + u sin a)`` with ``a
+    = p * f_i``, ``f_i = base^(-2i/dims)``. ``scaling`` rescales the frequencies: ``{"kind": "bands", factor, low, high, original}``
+    (:func:`banded_frequencies`) or ``{"kind": "ramp", factor, original, fast, slow}`` (:func:`ramped_frequencies`, which also multiplies cos and
+    sin by a constant). There is no table over all positions: each step computes cos and sin ``[tokens, dims / 2]`` for its own tokens once
+    (frequencies, products and functions in fp64, rounded once to fp32), shared by every layer with equal parameters, so no position limit
+    comes from here."""
 
-    halves = True
-    """Pairs are (i, i + dims / 2), not neighbours."""
+    halves = False
+    """Pairs are (i, i + dims / 2), not neighbours (2i, 2i + 1)."""
 
     def __init__(self, runtime: Runtime, *, dims: int, base: float, scaling: dict | None = None):
         if dims % 2 or dims <= 0:
@@ -120,14 +95,23 @@ class RotaryHalves(PositionEncoding):
         self.freq = torch.tensor(freq, dtype=torch.float64).to(runtime.device)
 
     def tables(self):
-        raise NotImplementedError("rope_halves has per-step angles (step_angles), not a table over all positions")
+        raise NotImplementedError("this encoding has per-step angles (step_angles), not a table over all positions")
 
     def step_angles(self, ctx: StepContext) -> tuple[torch.Tensor, torch.Tensor]:
-        key = ("rope_halves", self.dims, self.base, tuple(sorted(self.scaling.items())) if self.scaling else None)
+        # the angles do not depend on which entries form a pair: both layouts share them
+        key = ("step_angles", self.dims, self.base, tuple(sorted(self.scaling.items())) if self.scaling else None)
         if key not in ctx.shared:
-            cos, sin = ops.rotary_angles(ctx.positions, self.freq)
-            if self.magnitude != 1.0:
-                ops.scale_(cos, self.magnitude)
-                ops.scale_(sin, self.magnitude)
-            ctx.shared[key] = (cos, sin)
+            ctx.shared[key] = ops.rotary_angles(ctx.positions, self.freq, self.magnitude)
         return ctx.shared[key]
+
+
+@POSITION_ENCODINGS.register("rope_pairs")
+class RotaryPairs(StepAngles):
+    """Per-step angles for the interleaved layout: pair i is the entries 2i and 2i + 1."""
+
+
+@POSITION_ENCODINGS.register("rope_halves")
+class RotaryHalves(StepAngles):
+    """Per-step angles for the half-split layout: pair i is the entries i and i + dims / 2."""
+
+    halves = True
