@@ -1241,9 +1241,9 @@ def verorax_kernels(width: int, heads: int, kv_heads: int, head_dim: int, ff: in
     return rows
 
 
-def verorax_workload(args) -> int:
-    """The Verorax design beside Nidudra (the closest design: pairs of mixers, a recurrence, routed experts) and Qwen3 at equal sizes: whole-model
-    prefill and decode throughput at two sizes, and every kernel of its parts against its roofline beside the like kernel."""
+def designs_workload(args, workload: str, designs: dict, kernels) -> int:
+    """Designs at equal layer sizes beside each other: whole-model prefill and decode throughput at two sizes (``designs``: name -> function of the
+    sizes that gives a config), then ``kernels`` (a function of the larger size's numbers): every kernel against its roofline beside the like kernel."""
     import torch
 
     sizes = [("2048 wide, 8 layers", dict(width=2048, ff=8192, heads=16, kv_heads=4, head_dim=128, layers=8, vocab=32768)),
@@ -1251,23 +1251,191 @@ def verorax_workload(args) -> int:
     K, W = args.steps, max(args.warmup, 3)
     sampler = ClockSampler()
     sampler.start()
-    out = {"workload": "verorax", "dtype": "bf16", "data": "synthetic uniform token ids, random weights N(0, 0.02)", "steps": K, "warmup": W,
+    out = {"workload": workload, "dtype": "bf16", "data": "synthetic uniform token ids, random weights N(0, 0.02)", "steps": K, "warmup": W,
            "batch": 8, "context": args.context, "prefill_tokens": PREFILL_TOKENS, "peaks": peaks()[2], "sizes": []}
     for name, s in sizes:
-        qwen = {"architectures": ["Qwen3ForCausalLM"], "model_type": "qwen3", "hidden_size": s["width"], "intermediate_size": s["ff"],
-                "num_hidden_layers": s["layers"], "num_attention_heads": s["heads"], "num_key_value_heads": s["kv_heads"], "head_dim": s["head_dim"],
-                "rms_norm_eps": 1e-6, "rope_theta": 1000000.0, "vocab_size": s["vocab"], "tie_word_embeddings": False,
-                "max_position_embeddings": 8192}
         row = {"size": name}
-        for design, cfg in (("qwen3", qwen), ("nidudra", nidudra_config(**s)), ("verorax", verorax_config(**s))):
-            row[design] = design_throughput(cfg, s["vocab"], K, W, 8, args.context, PREFILL_TOKENS)
+        for design, config in designs.items():
+            row[design] = design_throughput(config(**s), s["vocab"], K, W, 8, args.context, PREFILL_TOKENS)
             torch.cuda.empty_cache()
         out["sizes"].append(row)
     last = sizes[-1][1]
-    out["kernels"] = verorax_kernels(last["width"], last["heads"], last["kv_heads"], last["head_dim"], last["ff"])
+    out["kernels"] = kernels(last["width"], last["heads"], last["kv_heads"], last["head_dim"], last["ff"])
     out["clocks"] = sampler.stop()
     print(json.dumps(out))
     return 0
+
+
+def qwen3_config(width: int, ff: int, heads: int, kv_heads: int, head_dim: int, layers: int, vocab: int) -> dict:
+    return {"architectures": ["Qwen3ForCausalLM"], "model_type": "qwen3", "hidden_size": width, "intermediate_size": ff, "num_hidden_layers": layers,
+            "num_attention_heads": heads, "num_key_value_heads": kv_heads, "head_dim": head_dim, "rms_norm_eps": 1e-6, "rope_theta": 1000000.0,
+            "vocab_size": vocab, "tie_word_embeddings": False, "max_position_embeddings": 8192}
+
+
+def verorax_workload(args) -> int:
+    """The Verorax design beside Nidudra (the closest design: pairs of mixers, a recurrence, routed experts) and Qwen3."""
+    return designs_workload(args, "verorax", {"qwen3": qwen3_config, "nidudra": nidudra_config, "verorax": verorax_config}, verorax_kernels)
+
+
+def finolix_config(width: int, ff: int, heads: int, kv_heads: int, head_dim: int, layers: int, vocab: int, experts: int = 16, top: int = 4) -> dict:
+    """A Finolix model of a real model's layer sizes: two residual streams; latent attention over the last 1,024 keys (rows of 192 + 64 entries,
+    queries through a latent of a quarter of the width, a sink per head) and gated attention (a quarter of each head rotated) take turns, with the
+    head sizes of the Qwen3 model beside it; the feed-forwards alternate between the square of relu, half as wide again as that model's gated
+    layer (two matrices instead of three: equal weights), and experts (``top`` of ``experts``, each an eighth of ``ff`` wide)."""
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top)}, "router": {"experts": experts, "top": top}}
+    scaling = {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": 64, "rot": {"dims": 64, "base": 10000.0, "scaling": scaling}, "vdim": head_dim, "kv_rank": 192,
+              "q_rank": width // 4, "scale": (head_dim + 64) ** -0.5, "mask": {"size": 1024}}
+    gated = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "rot": {"dims": head_dim // 4, "base": 100000.0}}
+    turn = (("latent_attention", latent), ("attention", gated))
+    return {"architecture": "Finolix", "norm": {"eps": 1e-6}, "vocab": vocab, "width": width, "streams": 2,
+            "layers": [{"type": turn[i % 2][0], "mixer": turn[i % 2][1], "mlp": (dense, moe)[i // 2 % 2]} for i in range(layers)]}
+
+
+def finolix_kernels(width: int, heads: int, kv_heads: int, head_dim: int, ff: int) -> list[dict]:
+    """Each kernel of the design alone, at one model size, beside the like kernel of the paths that were there before: device time (median, L2
+    flushed between calls), the bytes or FLOPs it has to move or do, and the fraction of the measured peak."""
+    import torch
+
+    from oxr_inference_b200 import ops
+    from oxr_inference_b200.parts.base import FEED_FORWARDS, Runtime
+
+    dev, bf = "cuda", torch.bfloat16
+    hbm_gbs, bf16_tflops, _ = peaks()
+    flush = torch.zeros(128 << 20, dtype=torch.float32, device=dev)
+    status = ops.new_status(dev)
+    rows = []
+
+    def put(name, like, fn, *, bytes_=None, flops=None):
+        ms = _time_ms(fn, flush=flush)
+        row = {"kernel": name, "like": like, "us": round(ms * 1e3, 1)}
+        if bytes_ is not None:
+            row.update(gb_s=round(bytes_ / (ms * 1e-3) / 1e9, 1), frac=round(bytes_ / (ms * 1e-3) / 1e9 / hbm_gbs, 4), bound="hbm")
+        else:
+            row.update(tflop_s=round(flops / (ms * 1e-3) / 1e12, 2), frac=round(flops / (ms * 1e-3) / 1e12 / bf16_tflops, 4), bound="tensor")
+        rows.append(row)
+
+    P, T, B, CTX = 16, 2048, 8, 2048
+    H, KV, D, L, R = heads, kv_heads, head_dim, 192, 64
+    QL, WINDOW = width // 4, 1024
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rand(*shape, dtype=bf, scale=1.0):
+        return (torch.randn(*shape, generator=g, device=dev) * scale).to(dtype)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    n_pages = B * (CTX // P) + T // P + 8
+    k_pool, v_pool, latent_pool = rand(n_pages, P, KV, D), rand(n_pages, P, KV, D), rand(n_pages, P, 1, L + R)
+    maps = ops.make_kv_maps(k_pool.unsqueeze(0), v_pool.unsqueeze(0), P)
+    cq, ck, cv = H * D, KV * D, KV * D
+    ones = torch.ones(D, device=dev)
+    cos_table = torch.ones(8192, D // 2, device=dev)
+    for name, q_lens, ctx_lens in (("prefill 2048", [T], [T]), ("decode b8", [1] * B, [CTX] * B)):
+        n, prefill, N = sum(q_lens), q_lens[0] > 1, len(q_lens)
+        cu = i32([0] + list(torch.tensor(q_lens).cumsum(0)))
+        req = torch.repeat_interleave(torch.arange(N, dtype=torch.int32), torch.tensor(q_lens)).to(dev)
+        pos = i32(list(range(T)) if prefill else [CTX - 1] * B)
+        slots = i32([(r * (CTX // P)) * P + (i if prefill else CTX - 1) for r, x in enumerate(q_lens) for i in range(x)])
+        table = torch.stack([torch.arange(r * (CTX // P), r * (CTX // P) + CTX // P + 1, dtype=torch.int32) % n_pages for r in range(N)]).to(dev).contiguous()
+        # ---- the streams
+        stream, w, x = torch.randn(n, width, device=dev), torch.ones(width, device=dev), rand(n, width)
+        put(f"add_rms_norm {name}", None, lambda: ops.add_rms_norm(x, stream, w, 1e-6), bytes_=n * width * (2 + 4 + 4 + 2))
+        put(f"norm_add_norm {name}", f"add_rms_norm {name}", lambda: ops.norm_add_norm(stream, x, w, 1e-6, w, 1e-6), bytes_=n * width * (2 + 4 + 4 + 2))
+        for S in (2, 4):
+            streams, mix, vec = torch.randn(n, S, width, device=dev), torch.eye(S, device=dev), torch.ones(S, device=dev)
+            update = dict(y=x, mix=mix, out_weights=vec, scale=w)
+            put(f"hyper_mix {name} ({S} streams: scale, mix, norm)", f"norm_add_norm {name}", lambda: ops.hyper_mix(streams, S, bf, then=(vec, w, 1e-6), **update),
+                bytes_=n * width * (2 + 2 + 8 * S))
+        put(f"hyper_mix {name} (4 streams into their sum)", f"norm_add_norm {name}", lambda: ops.hyper_mix(streams, 4, bf, **update), bytes_=n * width * (2 + 4 + 16))
+        # ---- between the products and attention
+        qkv = rand(n, cq + ck + cv, scale=0.5)
+        put(f"qk_norm_rope_store {name}", None,
+            lambda: ops.qk_norm_rope_store(qkv, ones, ones, cos_table, cos_table, pos, slots, k_pool, v_pool, H, KV, D, 1e-6, status), bytes_=n * (cq + ck + cv) * 4)
+        gproj, cos = rand(n, cq + ck + cv + H, scale=0.5), torch.ones(n, D // 8, device=dev)
+        put(f"head_prep {name} (q/k norm, a quarter of each head rotated, cache write)", f"qk_norm_rope_store {name}",
+            lambda: ops.head_prep(gproj, q_col0=0, k_col0=cq, v_col0=cq + ck, num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=D, norm="weighted", q_weight=ones,
+                                  k_weight=ones, cos=cos, sin=cos, k_pool=k_pool, v_pool=v_pool, slots=slots, n_requests=N, status=status, eps=1e-6,
+                                  req_of_token=req, cu_q=cu, state_slots=i32(list(range(N)))), bytes_=n * (cq + ck + cv) * 4)
+        down, q_lat = rand(n, QL + L + R), rand(n, H, D + R)
+        q_abs, cn, ang = torch.empty(n, H, L + R, dtype=bf, device=dev), torch.ones(L, device=dev), torch.ones(n, R // 2, device=dev)
+        for label, halves, like in (("half-split pairs, Verorax's", True, f"qk_norm_rope_store {name}"),
+                                    ("neighbouring pairs", False, f"latent_prep {name} (half-split pairs, Verorax's)")):
+            put(f"latent_prep {name} ({label})", like,
+                lambda: ops.latent_prep(latent_pool, down[:, QL:], L, R, cn, 1e-6, q_lat, H, D + R, D, q_abs, L + R, L, ang, ang, slots, status, halves=halves),
+                bytes_=n * ((L + R) * 4 + H * R * 4))
+
+        # ---- attention
+        def tiles_for(spec):
+            r_ = [r for r, x_ in enumerate(q_lens) if spec[1] <= x_ <= spec[2] for _ in range(0, x_, spec[0])]
+            t_ = [t0 for r, x_ in enumerate(q_lens) if spec[1] <= x_ <= spec[2] for t0 in range(0, x_, spec[0])]
+            return i32(r_ + [0]), i32(t_ + [0]), len(r_)
+
+        positions = range(T) if prefill else [CTX - 1] * B
+
+        def attention(label, like, kv_, k, v, *, tma, window=0, bytes_per_key=None, **extras):
+            width_ = k.shape[-1]
+            specs = ops.attention_tile_specs(H, kv_, width_, bf, P if tma else None)
+            q = rand(n, H, width_)
+            args = dict(tiles={spec: tiles_for(spec) for spec in specs}, cu_q=cu, ctx_lens=i32(ctx_lens), block_table=table, page_size=P, scale=D ** -0.5,
+                        window=window, kv_len_bound=max(ctx_lens), status=status, kv_maps=maps if tma else None, **extras)
+            seen = sum(min(p + 1, window) if window else p + 1 for p in positions)
+            put(label, like, lambda: ops.paged_attention(q, k, v, **args),
+                **(dict(flops=seen * 4 * H * width_) if prefill else dict(bytes_=seen * (bytes_per_key or kv_ * 4 * width_))))
+
+        tma_kind, cp_kind = ("tcgen05, TMA", "cp.async mma") if prefill else ("TMA split-KV", "cp.async split-KV")
+        attention(f"paged_attention {name} ({tma_kind})", None, KV, k_pool, v_pool, tma=True)
+        attention(f"paged_attention {name} ({cp_kind})", None, KV, k_pool, v_pool, tma=False)
+        sink = torch.zeros(H, device=dev)
+        latent = dict(tma=False, bytes_per_key=(L + R) * 2, sink=sink)
+        attention(f"latent attention {name} with a sink (Radapel's; {cp_kind})", f"paged_attention {name} ({cp_kind})", 1, latent_pool, latent_pool, **latent)
+        attention(f"latent attention {name} with a sink (last {WINDOW} keys; {cp_kind})", f"latent attention {name} with a sink (Radapel's; {cp_kind})", 1, latent_pool,
+                  latent_pool, window=WINDOW, **latent)
+        o, gates, pair = rand(n, H * D), rand(n, cq + ck + cv + H), rand(n, 2 * H * D)
+        put(f"silu_mul {name} ({H * D} columns)", None, lambda: ops.silu_mul(pair), bytes_=n * H * D * 6)
+        put(f"sigmoid_gate {name} (a gate per head, in place)", f"silu_mul {name} ({H * D} columns)",
+            lambda: ops.sigmoid_gate_(o, gates, cq + ck + cv, D, per_head=True), bytes_=n * H * D * 4)
+        # ---- the router
+        E, top = 16, 4
+        z, bias = torch.randn(n, E, device=dev), torch.zeros(E, device=dev)
+        put(f"route {name} (softmax of {E})", None, lambda: ops.route(z, top=top, groups=1, keep=1, scale=1.0, score="softmax", renormalize=False),
+            bytes_=n * (2 * E + 2 * top) * 4)
+        put(f"route {name} (biased, softmax over the {top} chosen)", f"route {name} (softmax of {E})",
+            lambda: ops.route(z, top=top, groups=1, keep=1, scale=1.0, score="chosen_softmax", bias=bias), bytes_=n * (2 * E + 2 * top) * 4)
+    # ---- the feed-forwards as a whole
+    rt = Runtime(device=torch.device(dev), dtype=bf, max_positions=1, status=status)
+
+    def built(kind, **params):
+        part = FEED_FORWARDS.build(kind, rt, hidden_size=width, **params)
+        for pname, info in part.parameters().items():
+            part.assign(pname, rand(*info.shape, scale=0.02))
+        part.finish_loading()
+        return part
+
+    E, top, ffe, ffd = 16, 4, ff // 8, ff * 3 // 2
+    swiglu, gelu, relu2 = built("swiglu", intermediate_size=ff), built("gelu_mlp", intermediate_size=ffd), built("relu2_mlp", intermediate_size=ffd)
+    common = dict(intermediate_size=ffe, experts=E, top=top, activation="silu_glu")
+    theirs, ours = built("routed_experts", score="softmax", renormalize=False, **common), built("routed_experts", score="chosen_softmax", router_bias=True, **common)
+    for n in (T, 256, B):
+        h = rand(n, width)
+        work = dict(flops=2 * n * width * 3 * ff) if n >= 256 else dict(bytes_=3 * ff * width * 2)
+        put(f"SiLU-gated feed-forward {n} rows ({ff})", None, lambda: swiglu.forward(h), **work)
+        put(f"GELU feed-forward {n} rows (two matrices, {ffd}; Vazepel's)", f"SiLU-gated feed-forward {n} rows ({ff})", lambda: gelu.forward(h), **work)
+        put(f"squared-relu feed-forward {n} rows ({ffd})", f"GELU feed-forward {n} rows (two matrices, {ffd}; Vazepel's)", lambda: relu2.forward(h), **work)
+        touched = E * (1 - (1 - top / E) ** n)
+        moe_work = dict(flops=2 * n * width * 3 * ffe * top) if n >= 256 else dict(bytes_=3 * width * 2 * touched * ffe)
+        put(f"routed experts {n} rows ({top} of {E} of {ffe}, softmax of all)", f"SiLU-gated feed-forward {n} rows ({ff})", lambda: theirs.forward(h), **moe_work)
+        put(f"routed experts {n} rows ({top} of {E} of {ffe}, biased, softmax over the chosen)", f"routed experts {n} rows ({top} of {E} of {ffe}, softmax of all)",
+            lambda: ours.forward(h), **moe_work)
+    ops.check_status(status)
+    return rows
+
+
+def finolix_workload(args) -> int:
+    """The Finolix design beside Verorax (the closest design: latent attention, gated attention, routed experts, a stream kept whole) and Qwen3."""
+    return designs_workload(args, "finolix", {"qwen3": qwen3_config, "verorax": verorax_config, "finolix": finolix_config}, finolix_kernels)
 
 
 def main() -> int:
@@ -1280,9 +1448,9 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="leave out batch 1 and 64 and the further points (quick runs)")
     ap.add_argument("--skip-serving", action="store_true", help="leave the two serving workloads out of `points`")
     ap.add_argument("--context", type=int, default=CONTEXT, help="tokens each request holds when the decode steps are timed")
-    ap.add_argument("--workload", default="decode", choices=("decode", "continuous", "chunked", "radapel", "bifusun", "vazepel", "nidudra", "verorax"),
+    ap.add_argument("--workload", default="decode", choices=("decode", "continuous", "chunked", "radapel", "bifusun", "vazepel", "nidudra", "verorax", "finolix"),
                     help="decode: the headline line (default); continuous / chunked: the two serving workloads, one line each; "
-                         "radapel / bifusun / vazepel / nidudra / verorax: that design beside Qwen3 (verorax: and Nidudra) at equal sizes, whole models and kernel by kernel")
+                         "radapel / bifusun / vazepel / nidudra / verorax / finolix: that design beside Qwen3 (verorax: and Nidudra, finolix: and Verorax) at equal sizes, whole models and kernel by kernel")
     args = ap.parse_args()
     if args.gpus != 1:
         print(f"this engine runs on one GPU; --gpus {args.gpus} is not supported")
@@ -1299,6 +1467,8 @@ def main() -> int:
         return nidudra_workload(args)
     if args.workload == "verorax":
         return verorax_workload(args)
+    if args.workload == "finolix":
+        return finolix_workload(args)
     if args.workload != "decode":
         return serving_workload(args.workload)
     K, W = args.steps, max(args.warmup, 3)
