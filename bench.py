@@ -1340,6 +1340,7 @@ def finolix_kernels(width: int, heads: int, kv_heads: int, head_dim: int, ff: in
         pos = i32(list(range(T)) if prefill else [CTX - 1] * B)
         slots = i32([(r * (CTX // P)) * P + (i if prefill else CTX - 1) for r, x in enumerate(q_lens) for i in range(x)])
         table = torch.stack([torch.arange(r * (CTX // P), r * (CTX // P) + CTX // P + 1, dtype=torch.int32) % n_pages for r in range(N)]).to(dev).contiguous()
+        state_slots = i32(list(range(N)))
         # ---- the streams
         stream, w, x = torch.randn(n, width, device=dev), torch.ones(width, device=dev), rand(n, width)
         put(f"add_rms_norm {name}", None, lambda: ops.add_rms_norm(x, stream, w, 1e-6), bytes_=n * width * (2 + 4 + 4 + 2))
@@ -1358,7 +1359,7 @@ def finolix_kernels(width: int, heads: int, kv_heads: int, head_dim: int, ff: in
         put(f"head_prep {name} (q/k norm, a quarter of each head rotated, cache write)", f"qk_norm_rope_store {name}",
             lambda: ops.head_prep(gproj, q_col0=0, k_col0=cq, v_col0=cq + ck, num_heads=H, num_kv_heads=KV, key_dim=D, value_dim=D, norm="weighted", q_weight=ones,
                                   k_weight=ones, cos=cos, sin=cos, k_pool=k_pool, v_pool=v_pool, slots=slots, n_requests=N, status=status, eps=1e-6,
-                                  req_of_token=req, cu_q=cu, state_slots=i32(list(range(N)))), bytes_=n * (cq + ck + cv) * 4)
+                                  req_of_token=req, cu_q=cu, state_slots=state_slots), bytes_=n * (cq + ck + cv) * 4)
         down, q_lat = rand(n, QL + L + R), rand(n, H, D + R)
         q_abs, cn, ang = torch.empty(n, H, L + R, dtype=bf, device=dev), torch.ones(L, device=dev), torch.ones(n, R // 2, device=dev)
         for label, halves, like in (("half-split pairs, Verorax's", True, f"qk_norm_rope_store {name}"),
