@@ -613,7 +613,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         raise KernelError(f"no tile list for long tiles of {long_rows} rows: the batch was cut for {sorted(tiles)}")
     s_req, s_tok, n_short = tiles[short]
     l_req, l_tok, n_long = tiles[long_]
-    seen = kv_len_bound if window <= 0 else min(kv_len_bound, window + keep_first + SHORT_MAX_TOKENS)     # keys a short tile can see
+    # the cp.async kernel deals out the keys that a short tile sees: no more than its window holds
+    seen = min(kv_len_bound, window + keep_first + SHORT_MAX_TOKENS) if masked and window > 0 else kv_len_bound
     splits, cut, part_o, part_ml, counters = _split_kv_plan(lib, n_short, num_heads, num_kv_heads, head_dim, seen, kv_maps is not None,
                                                             uneven, q.device)
     if masked:
